@@ -26,14 +26,15 @@ class KVLayerSpec:
     are then two device tensors, ``[layers, pages + 1, kv_heads, page_size, head_dim | value_dim]``.
     ``keep_first``: with a window, the sequence's first ``keep_first`` tokens stay readable as well.
     ``chunk``: a token reads only the keys of its own chunk of that many tokens (counted from the sequence's
-    first token); pages wholly before the current chunk are given back."""
+    first token); pages wholly before the current chunk are given back.  A tuple of chunk sizes: several layers read
+    this one's keys, each under chunks of its own; a page is given back when none of them needs it any more."""
 
     num_kv_heads: int
     head_dim: int
     window: int | None = None
     value_dim: int | None = None
     keep_first: int = 0
-    chunk: int | None = None
+    chunk: int | tuple[int, ...] | None = None
 
     @property
     def split(self) -> bool:
@@ -63,6 +64,26 @@ class LatentLayerSpec:
 class StateLayerSpec:
     shape: tuple[int, ...]
     dtype: str = "float32"
+
+
+def kept_for_readers(cache_id, own, others: list):
+    """The spec of cache layer ``cache_id`` that its writer (``own``) and further layers (``others``) read.  They agree
+    on heads and sizes; where their masks differ, what any of them may still read is kept."""
+    if all(spec == own for spec in others):
+        return own
+    specs = [own, *others]
+    if (not all(isinstance(s, KVLayerSpec) for s in specs)
+            or any((s.num_kv_heads, s.head_dim, s.value_dim or s.head_dim)
+                   != (own.num_kv_heads, own.head_dim, own.value_dim or own.head_dim) for s in specs)):
+        raise ValueError(f"a run entry reads cache layer {cache_id} whose layout differs from its own")
+    window = chunk = None
+    keep_first = 0
+    if all(s.chunk for s in specs):
+        chunk = tuple(sorted({c for s in specs for c in (s.chunk if isinstance(s.chunk, tuple) else (s.chunk,))}))
+        chunk = chunk[0] if len(chunk) == 1 else chunk
+    elif all(s.window for s in specs):
+        window, keep_first = max(s.window for s in specs), max(s.keep_first for s in specs)
+    return KVLayerSpec(own.num_kv_heads, own.head_dim, window, value_dim=own.value_dim, keep_first=keep_first, chunk=chunk)
 
 
 @dataclass(frozen=True)
@@ -156,7 +177,7 @@ class CacheLayout:
             return counts
         spent, open_bytes = 0, 0
         for i, gi in enumerate(self.paged_groups):
-            window = self.groups[gi].spec.window or self.groups[gi].spec.chunk  # the most keys a request holds
+            window = self.groups[gi].spec.reach  # the most keys a request holds
             if window:
                 kept = -(-self.groups[gi].spec.keep_first // page_size)
                 cap = max_num_seqs * (-(-(window + max_step_tokens) // page_size) + 2 + kept)
@@ -166,6 +187,6 @@ class CacheLayout:
                 open_bytes += per[i]
         if open_bytes:
             full = int((budget_bytes - spent) // open_bytes)
-            counts = [c if (self.groups[gi].spec.window or self.groups[gi].spec.chunk) else full
+            counts = [c if self.groups[gi].spec.reach else full
                       for c, gi in zip(counts, self.paged_groups)]
         return counts

@@ -44,19 +44,30 @@ class GroupSpec:
     kind: str
     window: int | None = None
     keep_first: int = 0  # a window group: the first tokens of a sequence that stay readable too
-    chunk: int | None = None  # a chunk group: the chunks' size
+    chunk: int | tuple[int, ...] | None = None  # a chunk group: the chunks' size (or those of several readers)
 
     def __post_init__(self) -> None:
         if self.kind not in ("full", "window", "chunk", "state"):
             raise ValueError(f"unknown cache group kind {self.kind!r}")
         if self.kind == "window" and (self.window is None or self.window < 1):
             raise ValueError("a window group needs window >= 1")
-        if self.kind == "chunk" and (self.chunk is None or self.chunk < 1):
+        if self.kind == "chunk" and (not self.chunks or min(self.chunks) < 1):
             raise ValueError("a chunk group needs chunk >= 1")
 
     @property
     def paged(self) -> bool:
         return self.kind != "state"
+
+    @property
+    def chunks(self) -> tuple[int, ...]:
+        if self.chunk is None:
+            return ()
+        return self.chunk if isinstance(self.chunk, tuple) else (self.chunk,)
+
+    @property
+    def reach(self) -> int | None:
+        """The most keys before a token that any of the group's layers reads (None: all)."""
+        return self.window or (max(self.chunks) if self.chunks else None)
 
 
 class PageAllocator:
@@ -235,7 +246,7 @@ class CacheManager:
             group = self.groups[gi]
             if group.kind == "chunk":
                 # the next query sits at position >= end and reads no key before the chunk that holds `end`
-                first_needed = end // group.chunk * group.chunk
+                first_needed = min(end // size * size for size in group.chunks)
                 kept_pages = 0
             elif group.kind == "window":
                 # the next query sits at position >= end and reads keys > end - window

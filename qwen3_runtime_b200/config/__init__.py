@@ -3,6 +3,7 @@ from .logesun_config import LogesunConfig
 from .medilix_config import MedilixConfig
 from .puladra_config import PuladraConfig
 from .tabisun_config import TabisunConfig
+from .pevazen_config import PevazenConfig
 from .model_config import ConfigError, Qwen3Config
 from .registry import (
     Architecture,
@@ -28,6 +29,7 @@ __all__ = [
     "MedilixConfig",
     "ModelSpec",
     "PartSpec",
+    "PevazenConfig",
     "PuladraConfig",
     "Qwen3Config",
     "TabisunConfig",

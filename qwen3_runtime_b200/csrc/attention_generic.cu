@@ -29,8 +29,9 @@ __global__ void paged_attention_generic_kernel(const T* __restrict__ q, int q_st
                                                long out_stride, int num_tokens, int nq, int nkv, int D, int Dv, int ps, float scale,
                                                int window, int keep_first, int has_sink, float sink,
                                                const T* __restrict__ gate, long gate_stride, int chunk,
-                                               float softcap) {
-  extern __shared__ float qs_all[];  // WARPS * D
+                                               float softcap, const float* __restrict__ turns, int turn_pairs,
+                                               int turn_pairing) {
+  extern __shared__ float qs_all[];  // WARPS * D (with turns: WARPS * max(D, Dv))
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long item = (long)blockIdx.x * WARPS + warp;
   if (item >= (long)num_tokens * nq) return;
@@ -39,7 +40,7 @@ __global__ void paged_attention_generic_kernel(const T* __restrict__ q, int q_st
   const int kvh = h / (nq / nkv);
   const int p = positions[t];
   const int* bt = block_table + (long)token_seq[t] * max_pages;
-  float* qs = qs_all + warp * D;
+  float* qs = qs_all + warp * (turns ? max(D, Dv) : D);
   const T* qrow = q + (long)t * q_stride + (long)h * D;
   for (int d = lane; d < D; d += 32) qs[d] = to_f32(qrow[d]);
   __syncwarp();
@@ -105,6 +106,23 @@ __global__ void paged_attention_generic_kernel(const T* __restrict__ q, int q_st
     for (int c = 0; c < 8; ++c) acc[c] *= corr;
   }
   const float inv = 1.f / l;
+  if (turns) {  // the sum of turned values is turned back by this token's angles
+    __syncwarp();
+#pragma unroll
+    for (int c = 0; c < 8; ++c)
+      if (lane + 32 * c < Dv) qs[lane + 32 * c] = acc[c];
+    __syncwarp();
+    const float* cs = turns + (long)t * 2 * turn_pairs;
+#pragma unroll
+    for (int c = 0; c < 8; ++c) {
+      const int d = lane + 32 * c;
+      if (d >= Dv || d >= 2 * turn_pairs) continue;
+      const bool first = turn_pairing ? (d & 1) == 0 : d < turn_pairs;  // the pair's first element
+      const int m = turn_pairing ? d >> 1 : (first ? d : d - turn_pairs);
+      const float other = qs[turn_pairing ? d ^ 1 : (first ? d + turn_pairs : d - turn_pairs)];
+      acc[c] = first ? acc[c] * cs[m] + other * cs[turn_pairs + m] : acc[c] * cs[m] - other * cs[turn_pairs + m];
+    }
+  }
   const T* grow = gate ? gate + (long)t * gate_stride + (long)h * Dv : nullptr;
 #pragma unroll
   for (int c = 0; c < 8; ++c) {
@@ -121,34 +139,38 @@ __global__ void paged_attention_generic_kernel(const T* __restrict__ q, int q_st
 // [pages, nkv, ps, D], values [pages, nkv, ps, Dv].  out: rows out_stride elements apart, head h at
 // column h*Dv.  window <= 0: none; keep_first counts only with a window; gate: rows gate_stride elements
 // apart, head h at column h*Dv, or null.  chunk <= 0: no chunked mask; softcap <= 0: scores as they are.
+// turns: null, or fp32 [num_tokens, 2, turn_pairs] (cos, then sin): the values in the cache are turned by their own
+// positions and a head's result is turned back by the token's angles (pairs (m, m + turn_pairs), or with
+// turn_pairing 1 (2m, 2m + 1)) before the gate.
 Q3_EXPORT int q3_paged_attention_generic(int dtype, const void* q, int q_stride, const void* kpages,
                                          const void* vpages, const int* block_table, int max_pages,
                                          const int* token_seq, const int* positions, void* out,
                                          long out_stride, int num_tokens, int nq, int nkv, int D, int Dv, int ps,
                                          float scale, int window, int keep_first, int has_sink, float sink,
                                          const void* gate, long gate_stride, int chunk, float softcap,
-                                         cudaStream_t stream) {
+                                         const float* turns, int turn_pairs, int turn_pairing, cudaStream_t stream) {
   if (!q || !kpages || !vpages || !block_table || !token_seq || !positions || !out) return Q3_ERR_ARGUMENT;
   if (nq < 1 || nkv < 1 || nq % nkv || ps < 1) return Q3_ERR_ARGUMENT;
   if (D < 1 || D > 256 || Dv < 1 || Dv > 256 || out_stride < (long)nq * Dv) return Q3_ERR_UNSUPPORTED;
   if (keep_first < 0 || (gate && gate_stride < (long)nq * Dv)) return Q3_ERR_ARGUMENT;
   if (chunk < 0 || softcap < 0.f || (chunk > 0 && keep_first > 0)) return Q3_ERR_ARGUMENT;
+  if (turns && (turn_pairs < 1 || 2 * turn_pairs > Dv || turn_pairing < 0 || turn_pairing > 1)) return Q3_ERR_ARGUMENT;
   if (window <= 0) keep_first = 0;
   if (num_tokens == 0) return Q3_OK;
   constexpr int WARPS = 4;
-  const size_t smem = (size_t)WARPS * D * sizeof(float);
+  const size_t smem = (size_t)WARPS * (turns && Dv > D ? Dv : D) * sizeof(float);
   const long items = (long)num_tokens * nq;
   const unsigned blocks = (unsigned)((items + WARPS - 1) / WARPS);
   if (dtype == Q3_DTYPE_F32)
     paged_attention_generic_kernel<float, WARPS><<<blocks, WARPS * 32, smem, stream>>>(
         (const float*)q, q_stride, (const float*)kpages, (const float*)vpages, block_table, max_pages,
         token_seq, positions, (float*)out, out_stride, num_tokens, nq, nkv, D, Dv, ps, scale, window, keep_first,
-        has_sink, sink, (const float*)gate, gate_stride, chunk, softcap);
+        has_sink, sink, (const float*)gate, gate_stride, chunk, softcap, turns, turn_pairs, turn_pairing);
   else if (dtype == Q3_DTYPE_BF16)
     paged_attention_generic_kernel<bf16, WARPS><<<blocks, WARPS * 32, smem, stream>>>(
         (const bf16*)q, q_stride, (const bf16*)kpages, (const bf16*)vpages, block_table, max_pages,
         token_seq, positions, (bf16*)out, out_stride, num_tokens, nq, nkv, D, Dv, ps, scale, window, keep_first,
-        has_sink, sink, (const bf16*)gate, gate_stride, chunk, softcap);
+        has_sink, sink, (const bf16*)gate, gate_stride, chunk, softcap, turns, turn_pairs, turn_pairing);
   else
     return Q3_ERR_ARGUMENT;
   return q3_launch_status();

@@ -360,3 +360,168 @@ Q3_EXPORT int q3_qk_norm_store(int dtype, void* proj, long row_stride, int nq, i
     return Q3_ERR_ARGUMENT;
   return e == cudaSuccess ? Q3_OK : Q3_ERR_LAUNCH;
 }
+
+// ---- rotations of a step's tokens, worked out once for all layers that turn by the same frequencies ----
+// turns [num_tokens, 2, n]: cos then sin of float(position) * inv_freq[m] (exact cosf / sinf).
+__global__ void turn_table_kernel(const int* __restrict__ positions, const float* __restrict__ inv_freq, int n,
+                                  float* __restrict__ turns, long total) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (idx >= total) return;
+  const long t = idx / n;
+  const int m = (int)(idx - t * n);
+  const float ang = (float)positions[t] * inv_freq[m];
+  turns[(2 * t) * n + m] = cosf(ang);
+  turns[(2 * t + 1) * n + m] = sinf(ang);
+}
+
+Q3_EXPORT int q3_turn_table(const int* positions, const float* inv_freq, int n, float* turns, int num_tokens,
+                            cudaStream_t stream) {
+  if (!positions || !inv_freq || !turns || n < 1) return Q3_ERR_ARGUMENT;
+  const long total = (long)num_tokens * n;
+  if (total == 0) return Q3_OK;
+  return launch_pdl(turn_table_kernel, dim3((unsigned)((total + 127) / 128)), dim3(128), 0, stream, positions, inv_freq,
+                    n, turns, total) == cudaSuccess
+             ? Q3_OK
+             : Q3_ERR_LAUNCH;
+}
+
+// ---- biases, rotation of q, k and (optionally) v, and the cache write, from a step's turn tables --------
+// A row of proj holds nq query heads of D from column 0, nkv key heads from k_start, nkv value heads of Dv from
+// v_start; bias (fp32, one number per column, or null) is added first.  The first 2 * qn elements of q and k heads
+// turn by qk_turns [T, 2, qn], the first 2 * vn of a value head by v_turns [T, 2, vn] (either may be null); the
+// sums are fp32, rounded once.  q is changed in place, k and v go to the token's rows of their pages.
+// A work unit is E pairs (or E elements that do not turn): E = 8 with 16-byte accesses (halves pairing, every
+// size a multiple of 8), else one.  Grid (tokens, blocks of units).
+template <typename T, int E>
+__device__ __forceinline__ void turn_unit(const T* __restrict__ x, const float* __restrict__ bias, T* __restrict__ dst,
+                                          int unit, int n, int pairing, const float* __restrict__ cs,
+                                          const float* __restrict__ sn) {
+  const int turning = n / E;
+  if (unit >= turning) {  // elements beyond the rotation
+    const int i = 2 * n + (unit - turning) * E;
+    if (E == 8) {
+      float a[8];
+      load8(x + i, a);
+      if (bias) {
+        float b[8];
+        load8(bias + i, b);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) a[e] += b[e];
+      }
+      store8(dst + i, a);
+    } else {
+      dst[i] = from_f32<T>(to_f32(x[i]) + (bias ? bias[i] : 0.f));
+    }
+    return;
+  }
+  if (E == 8) {
+    const int i = unit * 8;
+    float u[8], v[8], c[8], s[8];
+    load8(x + i, u);
+    load8(x + n + i, v);
+    load8(cs + i, c);
+    load8(sn + i, s);
+    if (bias) {
+      float b[8];
+      load8(bias + i, b);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) u[e] += b[e];
+      load8(bias + n + i, b);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] += b[e];
+    }
+    float a[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      a[e] = u[e] * c[e] - v[e] * s[e];
+      v[e] = v[e] * c[e] + u[e] * s[e];
+    }
+    store8(dst + i, a);
+    store8(dst + n + i, v);
+  } else {
+    const int i0 = pairing ? 2 * unit : unit, i1 = pairing ? i0 + 1 : unit + n;
+    const float u = to_f32(x[i0]) + (bias ? bias[i0] : 0.f), v = to_f32(x[i1]) + (bias ? bias[i1] : 0.f);
+    const float c = cs[unit], s = sn[unit];
+    dst[i0] = from_f32<T>(u * c - v * s);
+    dst[i1] = from_f32<T>(v * c + u * s);
+  }
+}
+
+template <typename T, int E>
+__global__ void turn_store_kernel(T* __restrict__ proj, long row_stride, int nq, int nkv, int D, int Dv, int k_start,
+                                  int v_start, const float* __restrict__ bias, const float* __restrict__ qk_turns, int qn,
+                                  const float* __restrict__ v_turns, int vn, int pairing,
+                                  const int* __restrict__ positions, const int* __restrict__ token_seq,
+                                  const int* __restrict__ block_table, int max_pages, T* __restrict__ kpages,
+                                  T* __restrict__ vpages, int ps, int write_kv) {
+  const int t = blockIdx.x;
+  int unit = blockIdx.y * blockDim.x + threadIdx.x;
+  const int qu = bias ? qn / E + (D - 2 * qn) / E : qn / E;  // without a bias what does not turn stays as it is
+  const int ku = qn / E + (D - 2 * qn) / E, vu = vn / E + (Dv - 2 * vn) / E;
+  if (unit >= nq * qu + (write_kv ? nkv * (ku + vu) : 0)) return;
+  pdl_wait();
+  pdl_launch_dependents();
+  T* row = proj + (long)t * row_stride;
+  const float* qc = qk_turns ? qk_turns + (long)t * 2 * qn : nullptr;
+  if (unit < nq * qu) {
+    const int h = unit / qu;
+    T* x = row + h * D;
+    turn_unit<T, E>(x, bias ? bias + h * D : nullptr, x, unit - h * qu, qn, pairing, qc, qc + qn);
+    return;
+  }
+  unit -= nq * qu;
+  const int p = positions[t];
+  if (p < 0 || p / ps >= max_pages) return;  // no page in the table for this position: write nothing
+  const int page = block_table[(long)token_seq[t] * max_pages + p / ps];
+  if (page < 0) return;
+  if (unit < nkv * ku) {
+    const int g = unit / ku;
+    const int col = k_start + g * D;
+    turn_unit<T, E>(row + col, bias ? bias + col : nullptr, kpages + (((long)page * nkv + g) * ps + p % ps) * D,
+                    unit - g * ku, qn, pairing, qc, qc + qn);
+    return;
+  }
+  unit -= nkv * ku;
+  const int g = unit / vu;
+  const int col = v_start + g * Dv;
+  const float* vc = v_turns ? v_turns + (long)t * 2 * vn : nullptr;
+  turn_unit<T, E>(row + col, bias ? bias + col : nullptr, vpages + (((long)page * nkv + g) * ps + p % ps) * Dv,
+                  unit - g * vu, vn, pairing, vc, vc + vn);
+}
+
+Q3_EXPORT int q3_turn_store(int dtype, void* proj, long row_stride, int nq, int nkv, int D, int Dv, int k_start,
+                            int v_start, const float* bias, const float* qk_turns, int qn, const float* v_turns, int vn,
+                            int pairing, const int* positions, const int* token_seq, const int* block_table,
+                            int max_pages, void* kpages, void* vpages, int ps, int num_tokens, int write_kv,
+                            cudaStream_t stream) {
+  if (!proj || !positions || nq < 1 || nkv < 1 || D < 1 || Dv < 1 || ps < 1) return Q3_ERR_ARGUMENT;
+  if (pairing < 0 || pairing > 1 || qn < 0 || vn < 0 || 2 * qn > D || 2 * vn > Dv) return Q3_ERR_ARGUMENT;
+  if ((qn > 0) != (qk_turns != nullptr) || (vn > 0) != (v_turns != nullptr)) return Q3_ERR_ARGUMENT;
+  if (write_kv && (!token_seq || !block_table || !kpages || !vpages || max_pages < 1)) return Q3_ERR_ARGUMENT;
+  if (num_tokens == 0) return Q3_OK;
+  const bool vec = (pairing == 0 || (qn == 0 && vn == 0)) && D % 8 == 0 && Dv % 8 == 0 && qn % 8 == 0 && vn % 8 == 0 &&
+                   k_start % 8 == 0 && v_start % 8 == 0 && row_stride % 8 == 0 && rk_aligned16(proj) &&
+                   rk_aligned16(bias) && rk_aligned16(qk_turns) && rk_aligned16(v_turns) && rk_aligned16(kpages) &&
+                   rk_aligned16(vpages);
+  const int E = vec ? 8 : 1;
+  const int units = nq * (bias ? (D - qn) / E : qn / E) + (write_kv ? nkv * ((D - qn) / E + (Dv - vn) / E) : 0);
+  if (units == 0) return Q3_OK;
+  const dim3 grid((unsigned)num_tokens, (unsigned)((units + 127) / 128));
+  if (grid.y > 65535) return Q3_ERR_UNSUPPORTED;
+  cudaError_t e;
+#define Q3_TURN_STORE(T, EE)                                                                                         \
+  e = launch_pdl(turn_store_kernel<T, EE>, grid, dim3(128), 0, stream, (T*)proj, row_stride, nq, nkv, D, Dv, k_start,  \
+                 v_start, bias, qk_turns, qn, v_turns, vn, pairing, positions, token_seq, block_table, max_pages,    \
+                 (T*)kpages, (T*)vpages, ps, write_kv)
+  if (dtype == Q3_DTYPE_F32) {
+    if (vec) Q3_TURN_STORE(float, 8); else Q3_TURN_STORE(float, 1);
+  } else if (dtype == Q3_DTYPE_BF16) {
+    if (vec) Q3_TURN_STORE(bf16, 8); else Q3_TURN_STORE(bf16, 1);
+  } else {
+    return Q3_ERR_ARGUMENT;
+  }
+#undef Q3_TURN_STORE
+  return e == cudaSuccess ? Q3_OK : Q3_ERR_LAUNCH;
+}

@@ -5,3 +5,4 @@ from . import logesun  # noqa: F401
 from . import puladra  # noqa: F401
 from . import medilix  # noqa: F401
 from . import tabisun  # noqa: F401
+from . import pevazen  # noqa: F401

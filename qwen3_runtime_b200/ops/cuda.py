@@ -123,7 +123,8 @@ _SIGNATURES = {
     "attention_generic": {
         "q3_paged_attention_generic": [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                        c_void_p, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                                       c_int, c_int, c_int, c_float, c_void_p, c_long, c_int, c_float, c_void_p],
+                                       c_int, c_int, c_int, c_float, c_void_p, c_long, c_int, c_float, c_void_p,
+                                       c_int, c_int, c_void_p],
         "q3_paged_attention_diff": [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                     c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
                                     c_float, c_float, c_float, c_void_p],
@@ -434,6 +435,68 @@ class CudaOps:
                    _ptr(out2), n, H, int(groups), float(eps), int(bool(write_resid)))
         return out
 
+    def sum_norm(self, out, weight, eps, *, resid, items, resid_out=None, points=None, num_points=0,
+                 depth_weights=None, rows=None, num_rows=None):
+        """Fold up to four sublayer outputs into the residual stream and norm the result (csrc/depth_norm.cu), float32
+        throughout.  ``items``: ``(value, norm_weight, norm_eps)`` each, ``value`` ``[rows, H]`` of the output's type or
+        fp32 partial sums ``[parts, rows, H]``; with a weight (fp32 ``[H]``) it is RMS-normalised before it is added.
+        ``v = resid + sum``; without ``depth_weights`` the stream becomes v, with them (fp32 ``[num_points + 1]``)
+        ``points[num_points] = v`` and the stream becomes ``sum_j depth_weights[j] * points[j]``, ``points`` fp32
+        ``[*, rows, H]``.  The stream goes to ``resid_out`` (None: nothing is written back); ``weight=None``: ``out``
+        gets the stream itself, rounded."""
+        H = resid.shape[-1]
+        n = out.shape[0] if num_rows is None else num_rows
+        if len(items) > 4:
+            raise KernelError("sum_norm: at most four outputs at a time")
+        if resid.dtype != torch.float32 or not resid.is_contiguous() or not out.is_contiguous() or out.shape[-1] != H:
+            raise KernelError("sum_norm: a dense float32 stream and dense output rows of its width")
+        if resid_out is not None and (resid_out.dtype != torch.float32 or not resid_out.is_contiguous()
+                                      or resid_out.shape != resid.shape):
+            raise KernelError("sum_norm: the stream is written to dense float32 rows")
+        if depth_weights is not None:
+            if (points is None or points.dtype != torch.float32 or not points.is_contiguous() or points.shape[2] != H
+                    or points.shape[1] != resid.shape[0] or points.shape[0] < num_points + 1):
+                raise KernelError("sum_norm: depth points are dense float32 [points, rows, width]")
+            if depth_weights.dtype != torch.float32 or depth_weights.numel() != num_points + 1:
+                raise KernelError(f"sum_norm: {depth_weights.numel()} depth weights for {num_points + 1} points")
+        flat = []
+        nbytes = 0
+        for value, w, e in items:
+            parts = stride = 0
+            if value.dim() == 3:
+                if value.dtype != torch.float32 or value.stride(2) != 1 or value.stride(1) != H or value.shape[2] != H:
+                    raise KernelError("sum_norm: partial sums are fp32 [parts, rows, H] with dense rows")
+                parts, stride = value.shape[0], value.stride(0)
+            elif value.dtype != out.dtype or not value.is_contiguous() or value.shape[-1] != H:
+                raise KernelError("sum_norm: an output to fold is dense [rows, H] of the output's type")
+            if w is not None and (w.dtype != torch.float32 or w.numel() != H or not w.is_contiguous()):
+                raise KernelError("sum_norm: norm weights are dense float32 vectors of the rows' width")
+            flat += [_ptr(value), parts, stride, _ptr(w), float(e)]
+            nbytes += 4 * parts if parts else out.element_size()
+        flat += [None, 0, 0, None, 0.0] * (4 - len(items))
+        if self.timing is not None:
+            depth = (4 * num_points + (4 if resid_out is not None else 0)) if depth_weights is not None else 0
+            # the stream's value is one of the points before the first average
+            own = 4 if depth_weights is None or resid.data_ptr() != points.data_ptr() else 0
+            self._costs(n * H * (own + nbytes + depth + (4 if resid_out is not None else 0) + out.element_size()))
+        self._call("depth_norm", "q3_sum_norm", "sum_norm", _dtype_code(out.dtype), len(items), *flat, _ptr(resid),
+                   _ptr(resid_out), _ptr(points) if depth_weights is not None else None,
+                   points.stride(0) if depth_weights is not None else 0, int(num_points), _ptr(depth_weights), _ptr(rows),
+                   _ptr(weight), _ptr(out), n, H, float(eps), int(resid_out is not None))
+        return out
+
+    def embed_norm(self, ids, table, weight, eps, out):
+        """``out[t] = table[ids[t]]`` divided by its root mean square, times ``weight`` (float32 rows)."""
+        T, W = out.shape
+        if out.dtype != torch.float32 or not out.is_contiguous() or not table.is_contiguous() or table.shape[1] != W \
+                or weight.dtype != torch.float32 or weight.numel() != W:
+            raise KernelError("embed_norm: dense float32 output rows and weight of the table's width")
+        if self.timing is not None:
+            self._costs(T * W * (4 + table.element_size()))
+        self._call("depth_norm", "q3_embed_norm", "embed_norm", _dtype_code(table.dtype), _ptr(ids), _ptr(table),
+                   table.shape[0], _ptr(weight), _ptr(out), T, W, float(eps))
+        return out
+
     def tanh_rows(self, x):
         """``x = tanh(x)`` in place (float32 math, one rounding)."""
         if not x.is_contiguous():
@@ -684,6 +747,96 @@ class CudaOps:
         if taps > 1:
             self._call("short_conv", "q3_conv_state_update", "conv_state_update", _dtype_code(x.dtype), _ptr(x),
                        x.stride(0), _ptr(conv_state), _ptr(cu_seqlens), _ptr(state_slots), taps, C, int(num_seqs))
+
+    # ---- gated delta rule (csrc/delta_state.cu) ------------------------------------------------------
+    def _delta_columns(self, x, conv_weight, ring, G, H, D, Dv, what):
+        C = 2 * G * D + H * Dv
+        taps = conv_weight.shape[0]
+        if x.stride(1) != 1 or x.shape[1] != C:
+            raise KernelError(f"{what}: rows of q, k and v heads with unit stride")
+        if conv_weight.dtype != torch.float32 or not conv_weight.is_contiguous() or conv_weight.shape[1] != C:
+            raise KernelError(f"{what}: a dense float32 weight [taps, channels]")
+        if taps > 1 and (ring is None or ring.dtype != torch.float32 or not ring.is_contiguous()
+                         or ring.shape[1:] != (taps, C)):
+            raise KernelError(f"{what}: the past inputs are a dense float32 ring [slots, taps, channels]")
+        if H % G or D > 256:
+            raise KernelError(f"{what}: whole groups of heads, key sizes up to 256")
+        return C, taps
+
+    def delta_rule(self, x, z, b, *, heads, kv_heads, dim, value_dim, conv_weight, ring, dt_bias, neg_a, state, positions,
+                   token_seq, cu_seqlens, state_slots, num_seqs, q_scale):
+        """The gated delta rule over a step's tokens (csrc/delta_state.cu): ``x`` ``[T, q heads | k heads | v heads]``
+        is convolved per channel (``conv_weight`` float32 ``[taps, C]``; past inputs in ``ring`` float32 ``[slots, taps,
+        C]``, brought up to date) and passed through silu, q and k become unit vectors (q times ``q_scale``), the decay
+        per head and key channel is ``exp(neg_a[h] * softplus(z + dt_bias))`` (``z`` float32 ``[T, H * D]``), the step
+        ``sigmoid(b)`` (``[T, H]``).  ``S <- decay * S; u = step * (v - S^T k); S <- S + k u^T; o = S^T q`` on the
+        float32 ``state`` ``[slots, H, D, Dv]``.  Returns float32 ``o`` ``[T, H, Dv]``."""
+        T = x.shape[0]
+        H, G, D, Dv = heads, kv_heads, dim, value_dim
+        C, taps = self._delta_columns(x, conv_weight, ring, G, H, D, Dv, "delta_rule")
+        if z.dtype != torch.float32 or not z.is_contiguous() or z.shape != (T, H * D):
+            raise KernelError("delta_rule: decay logits are dense float32 [tokens, heads * dim]")
+        if b.stride(1) != 1 or b.shape != (T, H) or b.dtype != x.dtype:
+            raise KernelError("delta_rule: one step logit per token and head, of the activations' type")
+        if state.dtype != torch.float32 or state.shape[1:] != (H, D, Dv) or not state.is_contiguous():
+            raise KernelError("delta_rule: the state is dense float32 [slots, H, D, Dv]")
+        dev = x.device
+        qn = torch.empty((T, G, D), dtype=torch.float32, device=dev)
+        kn = torch.empty_like(qn)
+        vc = torch.empty((T, H, Dv), dtype=x.dtype, device=dev)
+        g = torch.empty((T, H, D), dtype=torch.float32, device=dev)
+        beta = torch.empty((T, H), dtype=torch.float32, device=dev)
+        out = torch.empty((T, H, Dv), dtype=torch.float32, device=dev)
+        e = x.element_size()
+        if self.timing is not None:
+            self._costs(T * (C * e + 8 * G * D + H * Dv * e + 8 * H * D))
+        self._call("delta_state", "q3_delta_prepare", "delta_prepare", _dtype_code(x.dtype), _ptr(x), x.stride(0),
+                   _ptr(conv_weight), taps, _ptr(ring) if taps > 1 else None, _ptr(positions), _ptr(token_seq),
+                   _ptr(cu_seqlens), _ptr(state_slots), _ptr(z), _ptr(dt_bias), _ptr(neg_a), _ptr(b), b.stride(0),
+                   float(q_scale), _ptr(qn), _ptr(kn), _ptr(vc), _ptr(g), _ptr(beta), T, G, H, D, Dv)
+        if taps > 1:
+            self._call("delta_state", "q3_ring_update", "ring_update", _dtype_code(x.dtype), _ptr(x), x.stride(0),
+                       _ptr(ring), _ptr(positions), _ptr(cu_seqlens), _ptr(state_slots), taps, C, int(num_seqs))
+        if self.timing is not None:
+            self._costs(2 * num_seqs * H * D * Dv * 4 + T * (8 * G * D + H * Dv * (e + 4) + 4 * H * D),
+                        7.0 * T * H * D * Dv)
+        self._call("delta_state", "q3_delta_scan", "delta_scan", _dtype_code(x.dtype), _ptr(qn), _ptr(kn), _ptr(vc),
+                   _ptr(g), _ptr(beta), _ptr(state), _ptr(cu_seqlens), _ptr(state_slots), _ptr(out), int(num_seqs), G, H,
+                   D, Dv)
+        return out
+
+    def delta_step_ok(self, dim: int, value_dim: int) -> bool:
+        """Whether :meth:`delta_step` takes heads of these sizes."""
+        return dim <= 256 and value_dim <= 256 and dim * max(32, 1 << (value_dim - 1).bit_length()) <= 16384
+
+    def delta_step(self, x, low_a, low_g, b, out, *, heads, kv_heads, dim, value_dim, conv_weight, ring, a2, g2, dt_bias,
+                   neg_a, norm_weight, eps, state, positions, cu_seqlens, state_slots, num_seqs, q_scale):
+        """:meth:`delta_rule` for a step in which every sequence brings one token, with what stands before and after it
+        in one kernel: the decay logits are ``low_a @ a2^T``, and ``out`` gets each head's o divided by its root mean
+        square (``eps``), times ``norm_weight`` (float32 ``[Dv]``) and ``sigmoid(low_g @ g2^T)``.  ``x``, ``low_a``,
+        ``low_g`` and ``b`` are columns of one product."""
+        H, G, D, Dv = heads, kv_heads, dim, value_dim
+        C, taps = self._delta_columns(x, conv_weight, ring, G, H, D, Dv, "delta_step")
+        for y in (low_a, low_g, b):
+            if y.stride(1) != 1 or y.stride(0) != x.stride(0) or y.dtype != x.dtype:
+                raise KernelError("delta_step: x, the low-rank rows and the step logits are columns of one product")
+        if state.dtype != torch.float32 or state.shape[1:] != (H, D, Dv) or not state.is_contiguous():
+            raise KernelError("delta_step: the state is dense float32 [slots, H, D, Dv]")
+        if (a2.shape != (H * D, low_a.shape[1]) or g2.shape != (H * Dv, low_g.shape[1]) or not a2.is_contiguous()
+                or not g2.is_contiguous() or a2.dtype != x.dtype or g2.dtype != x.dtype):
+            raise KernelError("delta_step: dense second low-rank products of the activations' type")
+        if out.stride(1) != 1 or out.dtype != x.dtype or out.shape[1] != H * Dv:
+            raise KernelError("delta_step: the output is [tokens, heads * value_dim] of the activations' type")
+        if self.timing is not None:
+            e = x.element_size()
+            self._costs(num_seqs * (2 * H * D * Dv * 4 + (C + H * Dv) * e + C * (taps + 1) * 4)
+                        + (a2.numel() + g2.numel()) * e, 7.0 * num_seqs * H * D * Dv)
+        self._call("delta_state", "q3_delta_step", "delta_step", _dtype_code(x.dtype), _ptr(x), x.stride(0),
+                   _ptr(conv_weight), taps, _ptr(ring) if taps > 1 else None, _ptr(positions), _ptr(cu_seqlens),
+                   _ptr(state_slots), _ptr(low_a), _ptr(low_g), _ptr(a2), a2.shape[1], _ptr(g2), g2.shape[1],
+                   _ptr(dt_bias), _ptr(neg_a), _ptr(b), float(q_scale), _ptr(state), _ptr(norm_weight), float(eps),
+                   _ptr(out), out.stride(0), int(num_seqs), G, H, D, Dv)
+        return out
 
     # ---- attention through a latent (csrc/latent_attention.cu, csrc/head_gemm.cu) ---------------
     def latent_norm_rope_store(self, down, *, q_rank, kv_rank, rot_dim, q_weight, kv_weight, eps, inv_freq, positions,
@@ -986,11 +1139,51 @@ class CudaOps:
                    _ptr(positions), _ptr(token_seq), _ptr(block_table), max_pages,
                    _ptr(k_pages), _ptr(v_pages), page_size, T, int(bool(write_kv)))
 
+    def turn_table(self, positions, inv_freq):
+        """float32 ``[T, 2, n]``: cos and sin of ``position * inv_freq`` for every token of the step."""
+        T, n = positions.shape[0], inv_freq.numel()
+        out = torch.empty((T, 2, n), dtype=torch.float32, device=positions.device)
+        if inv_freq.dtype != torch.float32 or not inv_freq.is_contiguous():
+            raise KernelError("turn_table: dense float32 frequencies")
+        if self.timing is not None:
+            self._costs(out.numel() * 4)
+        self._call("rope_kv", "q3_turn_table", "turn_table", _ptr(positions), _ptr(inv_freq), n, _ptr(out), T)
+        return out
+
+    def turn_store(self, proj, *, num_heads, num_kv_heads, head_dim, value_dim, k_start, v_start, bias, qk_turns,
+                   value_turns, positions, token_seq, block_table, k_pages, v_pages, page_size, write_kv,
+                   pairing="half"):
+        """Biases, rotation and the cache write of a step's q, k and v heads (csrc/rope_kv.cu): ``bias`` (float32, one
+        number per column of ``proj``, or None) is added, q and k turn by ``qk_turns`` and, if given, v by
+        ``value_turns`` (:meth:`turn_table`; pairs of the leading elements as ``pairing`` says).  q is changed in
+        place; with ``write_kv=False`` only q is worked on."""
+        T = proj.shape[0]
+        if proj.stride(1) != 1:
+            raise KernelError("turn_store: unit-stride rows")
+        if bias is not None and (bias.dtype != torch.float32 or bias.numel() < proj.shape[1] or not bias.is_contiguous()):
+            raise KernelError("turn_store: a dense float32 bias, one number per column")
+        for turns in (qk_turns, value_turns):
+            if turns is not None and (turns.dtype != torch.float32 or not turns.is_contiguous()
+                                      or turns.shape[:2] != (T, 2)):
+                raise KernelError("turn_store: turn tables are dense float32 [tokens, 2, pairs]")
+        if self.timing is not None:
+            cols = num_heads * head_dim + (num_kv_heads * (head_dim + value_dim) if write_kv else 0)
+            self._costs(2 * T * cols * proj.element_size())
+        self._call("rope_kv", "q3_turn_store", "turn_store", _dtype_code(proj.dtype), _ptr(proj), proj.stride(0), num_heads,
+                   num_kv_heads, head_dim, value_dim, int(k_start), int(v_start), _ptr(bias), _ptr(qk_turns),
+                   qk_turns.shape[2] if qk_turns is not None else 0, _ptr(value_turns),
+                   value_turns.shape[2] if value_turns is not None else 0, self.PAIRINGS[pairing], _ptr(positions),
+                   _ptr(token_seq), _ptr(block_table), block_table.shape[1] if block_table is not None else 0,
+                   _ptr(k_pages), _ptr(v_pages), page_size, T, int(bool(write_kv)))
+
     # ---- attention --------------------------------------------------------------------
     def paged_attention(self, q, q_stride, *, num_heads, num_kv_heads, head_dim, k_pages, v_pages, block_table,
                         token_seq, positions, out, page_size, scale, window, step=None, decode_slices=None,
-                        value_dim=None, keep_first=0, sink=None, gate=None, chunk=None, softcap=None):
-        """Causal attention of every token of the step over its sequence's pages.  ``chunk``: position p sees
+                        value_dim=None, keep_first=0, sink=None, gate=None, chunk=None, softcap=None, value_turns=None,
+                        pairing="half"):
+        """Causal attention of every token of the step over its sequence's pages.  ``value_turns``
+        (:meth:`turn_table`): the cached values are turned by their own positions and a head's result is turned back
+        by its token's angles (pairs as ``pairing`` says).  ``chunk``: position p sees
         keys from ``floor(p / chunk) * chunk`` on only.  ``softcap``: scores become ``softcap * tanh(score /
         softcap)`` after the scale.  ``value_dim``:
         values have a size of their own (``v_pages`` ``[pages, kv heads, page, value_dim]``); ``out`` may
@@ -1007,8 +1200,11 @@ class CudaOps:
         dense = out.stride(0) == num_heads * Dv and Dv == head_dim
         extras = dict(keep_first=keep_first, sink=sink, gate=gate)
         chunk, softcap = int(chunk or 0), float(softcap or 0.0)
-        if chunk:
-            dense = False  # the specialised kernels know no chunks: the general kernel
+        if value_turns is not None and (value_turns.dtype != torch.float32 or not value_turns.is_contiguous()
+                                        or value_turns.shape[:2] != (T, 2)):
+            raise KernelError("paged_attention: value turns are dense float32 [tokens, 2, pairs]")
+        if chunk or value_turns is not None:
+            dense = False  # those specialised kernels know no chunks and no turned values
         if softcap:
             plain = False  # the tcgen05 kernel knows no capped scores; the other specialised kernels do
             extras["softcap"] = softcap
@@ -1080,7 +1276,8 @@ class CudaOps:
                   block_table.shape[1], _ptr(token_seq), _ptr(positions), _ptr(out), out.stride(0), T, num_heads,
                   num_kv_heads, head_dim, Dv, page_size, float(scale), int(window or 0), int(keep_first or 0),
                   int(sink is not None), float(sink or 0.0), _ptr(gate), gate.stride(0) if gate is not None else 0,
-                  chunk, softcap)
+                  chunk, softcap, _ptr(value_turns), value_turns.shape[2] if value_turns is not None else 0,
+                  self.PAIRINGS[pairing])
         return out
 
     def differential_attention(self, q, q_stride, *, num_heads, num_kv_heads, map_dim, value_dim, k_pages, v_pages,

@@ -146,6 +146,17 @@ def build_part(category: str, spec: PartSpec, ctx: BuildContext) -> Part:
     return factory(spec, ctx)
 
 
+@dataclass
+class Addend:
+    """One sublayer output that is still to be added to the residual sum: ``value`` ``[tokens, hidden]`` in the compute
+    dtype or float32 partial sums ``[parts, tokens, hidden]``; with ``norm_weight`` (float32 ``[hidden]``) it is
+    RMS-normalised first."""
+
+    value: torch.Tensor
+    norm_weight: torch.Tensor | None = None
+    norm_eps: float = 0.0
+
+
 class ResidualStream:
     """The residual sum of a step, kept in float32, plus what has not been added yet.
 
@@ -165,6 +176,11 @@ class ResidualStream:
     ``pending_more``: a second sublayer output ``[tokens, hidden]`` in the compute dtype that is added
     together with ``pending`` (a block whose mixer and feed-forward read the same input).
 
+    ``addends``: several outputs (:class:`Addend`) that the next norm folds in at once, in place of ``pending``.
+    ``points`` float32 ``[n, tokens, hidden]`` with ``num_points`` rows filled: the stream's values between the
+    layers of a model whose layers read an average over the depth.  ``depth_weights`` (float32 ``[num_points + 1]``):
+    the next norm stores the folded sum as a further point and the sum becomes the weighted sum of all points.
+
     A stream may also be started by an ``embedding`` part (:meth:`started`): ``resid`` then holds the
     embedding output already, and ``source_pair`` (if the model asked for it) is a buffer
     ``[tokens, 2 * hidden]`` in the compute dtype whose right half holds the embedding output, the left
@@ -183,6 +199,10 @@ class ResidualStream:
         self.pending_norm: tuple[torch.Tensor, float] | None = None
         self.add_source = False
         self.add_vector: torch.Tensor | None = None
+        self.addends: list[Addend] = []
+        self.points: torch.Tensor | None = None
+        self.num_points = 0
+        self.depth_weights: torch.Tensor | None = None
 
     @classmethod
     def started(cls, resid: torch.Tensor, source_pair: torch.Tensor | None = None) -> "ResidualStream":

@@ -7,11 +7,14 @@ x += norm_b(ff(norm(x))), the feed-forward being optional.
 ``parallel_norms``: mixer and feed-forward read the same stream through a norm each and are added
 together, x += mixer(norm_a(x)) + ff(norm_b(x)); the feed-forward is optional.
 ``output_norm``: the sublayers read the stream itself and only their outputs are normed,
-x += norm_a(mixer(x)); x += norm_b(ff(x)); the feed-forward is optional."""
+x += norm_a(mixer(x)); x += norm_b(ff(x)); the feed-forward is optional.
+``shared_norm``: mixer and feed-forward read one norm's output and are added together, x += mixer(h) + ff(h) with
+h = norm(x); the feed-forward is optional.  With ``depth_points`` the block owns that many weights, and what goes on
+is their weighted sum of the embedding output and the results of all layers so far."""
 
 from __future__ import annotations
 
-from .base import BuildContext, Part, ResidualStream, StepContext, build_part, register_part
+from .base import Addend, BuildContext, ParamSpec, Part, ResidualStream, StepContext, build_part, register_part
 
 
 class PreNormBlock(Part):
@@ -279,7 +282,74 @@ class OutputNormBlock(Part):
             stream.pending_norm = self.feed_forward_out_norm.pending_scale()
 
 
+class SharedNormBlock(Part):
+    """x += mixer(h) + ff(h), h = norm(x).  The outputs (a mixer may give several, each with a norm of its own) are
+    left on the stream as addends; whichever norm reads the stream next folds them in one kernel, which also takes
+    the average over the depth when the block has weights for it."""
+
+    category = "block"
+
+    def __init__(self, spec, ctx: BuildContext):
+        super().__init__(spec, ctx)
+        self.mixer = build_part("mixer", spec["mixer"], ctx)
+        self.norm = build_part("norm", spec["norm"], ctx)
+        self.children = {spec.get("mixer_prefix", "mixer."): self.mixer, spec.get("norm_prefix", "norm."): self.norm}
+        self.feed_forward = None
+        if spec.get("feed_forward") is not None:
+            self.feed_forward = build_part("feed_forward", spec["feed_forward"], ctx)
+            self.children[spec.get("feed_forward_prefix", "feed_forward.")] = self.feed_forward
+        self.depth_points = int(spec.get("depth_points") or 0)
+        self.depth_name = str(spec.get("depth_name", "depth_weights"))
+        self.depth_weights = None
+        self.entry_norm = self.norm
+        # the kernel that folds addends adds partial sums in any case
+        self.mixer.partial_sums_ok = True
+        if self.feed_forward is not None:
+            self.feed_forward.partial_sums_ok = True
+        self._owners = {prefix + name: (part, name) for prefix, part in self.children.items()
+                        for name in part.param_specs()}
+
+    def param_specs(self):
+        specs = {full: part.param_specs()[name] for full, (part, name) in self._owners.items()}
+        if self.depth_points:
+            specs[self.depth_name] = ParamSpec((self.depth_points,), "vector")
+        return specs
+
+    def load(self, tensors):
+        per_part: dict[int, dict] = {}
+        for full, (part, name) in self._owners.items():
+            per_part.setdefault(id(part), {})[name] = tensors[full]
+        for part in self.children.values():
+            part.load(per_part.get(id(part), {}))
+        if self.depth_points:
+            self.depth_weights = tensors[self.depth_name].contiguous()
+
+    def kernel_groups(self):
+        return ["depth_norm", *[g for part in self.children.values() for g in part.kernel_groups()]]
+
+    def step_choosers(self):
+        return {name: fn for part in self.children.values() for name, fn in part.step_choosers().items()}
+
+    def cache_spec(self):
+        return self.mixer.cache_spec()
+
+    def position_limit(self):
+        limits = [n for n in (part.position_limit() for part in self.children.values()) if n is not None]
+        return min(limits) if limits else None
+
+    def forward(self, stream: ResidualStream, step: StepContext, cache) -> None:
+        h = self.norm.add_norm(stream)
+        y = self.mixer.forward(h, step, cache)
+        addends = list(y) if isinstance(y, (list, tuple)) else [Addend(y)]
+        if self.feed_forward is not None:
+            addends.append(Addend(self.feed_forward.forward(h, step)))
+        stream.addends = addends
+        if self.depth_points:
+            stream.depth_weights = self.depth_weights
+
+
 register_part("block", "output_norm", OutputNormBlock)
+register_part("block", "shared_norm", SharedNormBlock)
 register_part("block", "pre_norm", PreNormBlock)
 register_part("block", "parallel_norms", ParallelNormsBlock)
 register_part("block", "sandwich_norm", SandwichNormBlock)

@@ -24,7 +24,7 @@ import torch
 
 from ..cache.layout import StateLayerSpec
 from ..config.spec import PartSpec
-from .base import BuildContext, ParamSpec, Part, StepContext, build_part, register_part
+from .base import Addend, BuildContext, ParamSpec, Part, StepContext, build_part, register_part
 
 
 def heads_view(rows: torch.Tensor, start: int, heads: int, size: int) -> torch.Tensor:
@@ -204,7 +204,10 @@ class ParallelMixer(Part):
     the norm adds the planes (no kernel adds the branches up, and every branch has a dense buffer,
     which the specialised attention kernels want); else the branches write into their columns of one
     buffer and the projections, laid side by side, multiply that buffer once.
-    ``branches``: ``[(prefix, PartSpec of a BranchMixer, scale), ...]``."""
+    ``branches``: ``[(prefix, PartSpec of a BranchMixer, scale), ...]``.
+    ``out_norms``: ``[(weight name, eps), ...]``, one per branch: every branch's output is RMS-normalised over the
+    model's width with a weight of its own before it is added (its scale goes into that weight); the mixer then
+    answers with the outputs side by side (:class:`Addend`), which the next norm's kernel norms and adds."""
 
     category = "mixer"
 
@@ -217,16 +220,25 @@ class ParallelMixer(Part):
                 raise ValueError(f"mixer {part_spec.kind!r} cannot run as a branch of a parallel mixer")
             self.branches.append((str(prefix), part, float(scale)))
         self._owners = {prefix + name: (part, name) for prefix, part, _ in self.branches for name in part.param_specs()}
+        self.out_norms = [(str(name), float(eps)) for name, eps in spec.get("out_norms") or ()]
+        if self.out_norms and len(self.out_norms) != len(self.branches):
+            raise ValueError("parallel: one output norm per branch, or none")
+        self.hidden_size = int(spec["hidden_size"]) if self.out_norms else 0
         self.in_weight = self.o_weight = None
+        self.out_norm_weights: list[torch.Tensor] = []
         self.in_starts: list[int] = []
         self.out_starts: list[int] = []
 
     def param_specs(self):
-        return {full: part.param_specs()[name] for full, (part, name) in self._owners.items()}
+        specs = {full: part.param_specs()[name] for full, (part, name) in self._owners.items()}
+        specs.update({name: ParamSpec((self.hidden_size,), "vector") for name, _eps in self.out_norms})
+        return specs
 
     def load(self, tensors):
         for prefix, part, _ in self.branches:
             part.load({name: tensors[prefix + name] for name in part.param_specs()})
+        self.out_norm_weights = [(tensors[name].float() * scale).contiguous()
+                                 for (name, _eps), (_p, _part, scale) in zip(self.out_norms, self.branches)]
         self.in_weight, self.in_starts = _pad_rows([part.input_weight() for _, part, _ in self.branches])
         self.o_weight = None  # the projections side by side; made when first needed
         self.in_sizes = [part.input_weight().shape[0] for _, part, _ in self.branches]
@@ -252,6 +264,14 @@ class ParallelMixer(Part):
     def forward(self, h: torch.Tensor, step: StepContext, cache) -> torch.Tensor:
         proj = self.ops.linear(h, self.in_weight)
         T = h.shape[0]
+        if self.out_norms:
+            addends = []
+            for i, ((_, part, _scale), a, n, view) in enumerate(zip(self.branches, self.in_starts, self.in_sizes, cache)):
+                ctx = torch.empty((T, part.context_size()), dtype=h.dtype, device=h.device)
+                part.context(proj[:, a:a + n], step, view, ctx, 1.0)
+                y = self.ops.linear(ctx, part.output_weight(), partial_sums=True)
+                addends.append(Addend(y, self.out_norm_weights[i], self.out_norms[i][1]))
+            return addends
         if self.partial_sums_ok:
             planes = torch.empty((len(self.branches), T, self.in_weight.shape[1]), dtype=torch.float32, device=h.device)
             for i, ((_, part, scale), a, n, view) in enumerate(zip(self.branches, self.in_starts, self.in_sizes, cache)):

@@ -8,7 +8,7 @@ from __future__ import annotations
 
 import torch
 
-from ..cache.layout import CacheLayout
+from ..cache.layout import CacheLayout, kept_for_readers
 from ..config.spec import ModelSpec
 from .base import BuildContext, ParamSpec, ResidualStream, StepContext, build_part
 from .norm import fold_stream
@@ -38,6 +38,13 @@ class DecoderModel:
             block = self.blocks[index]
             if hasattr(block, "exit_to") and all(n is not None for n in norms):
                 block.exit_to(norms)
+        # layers that read an average over the depth: every run adds a point behind the embedding output
+        averaging = [getattr(self.blocks[run.block], "depth_points", 0) for run in spec.order]
+        self.num_points = len(averaging) + 1 if any(averaging) else 0
+        if self.num_points:
+            if self.embedding is None or averaging != list(range(2, self.num_points + 1)):
+                raise ValueError("averages over the depth: an embedding part, and the run in place i (from 0) weighs i + 2 "
+                                 f"points (the runs weigh {averaging})")
         self.choosers: dict = {}
         for block in self.blocks:
             self.choosers.update(block.step_choosers())
@@ -106,15 +113,17 @@ class DecoderModel:
 
     # ---- cache ------------------------------------------------------------------------
     def cache_layout(self) -> CacheLayout:
-        specs = {}
+        specs, readers = {}, {}
         if self.embedding is not None:  # what the embedding keeps per request (the previous token)
             specs[EMBEDDING_CACHE] = self.embedding.cache_spec()
         for run in self.spec.order:
             if run.writes:
                 specs[run.cache] = self.blocks[run.block].cache_spec()
         for run in self.spec.order:
-            if not run.writes and specs[run.cache] != self.blocks[run.block].cache_spec():
-                raise ValueError(f"a run entry reads cache layer {run.cache} whose layout differs from its own")
+            if not run.writes:
+                readers.setdefault(run.cache, []).append(self.blocks[run.block].cache_spec())
+        for cache, others in readers.items():  # what is kept has to serve every reader's mask
+            specs[cache] = kept_for_readers(cache, specs[cache], others)
         return CacheLayout(specs)
 
     def step_choices(self, kv_lens: list[int]) -> dict:
@@ -127,7 +136,8 @@ class DecoderModel:
         ``step.logit_rows`` (None when no logits are wanted)."""
         s = self.spec
         if self.embedding is not None:
-            stream = self.embedding.start(step, storage.view(EMBEDDING_CACHE), keep_source=self.keeps_source)
+            stream = self.embedding.start(step, storage.view(EMBEDDING_CACHE), keep_source=self.keeps_source,
+                                          num_points=self.num_points)
         else:
             stream = ResidualStream(step.num_tokens, s.hidden_size, ids=step.token_ids, table=self.embed)
         for run in s.order:

@@ -3,6 +3,7 @@
 is the deviation from this value, which is added to it when it is loaded (y = ... * (offset + w)).
 ``groups`` > 1: a row is cut into that many equal consecutive parts and each is divided by its own root
 mean square (the weight still spans the whole row).
+``scalar``: the stored weight is one number for all coordinates (a tensor without dimensions).
 ``layernorm``: y = (x - mean(x)) * rsqrt(mean((x - mean(x))^2) + eps) * w, a weight and no bias; the same part
 with the mean taken off first (the same kernels with their ``center`` flags)."""
 
@@ -26,6 +27,7 @@ class RMSNorm(Part):
         self.weight_name = str(spec.get("weight_name", "weight"))
         self.weight_offset = float(spec.get("weight_offset", 0.0))
         self.groups = int(spec.get("groups") or 1)
+        self.scalar = bool(spec.get("scalar", False))
         if self.groups < 1 or self.size % self.groups:
             raise ValueError(f"rmsnorm: {self.size} elements do not split into {self.groups} equal groups")
         if self.center and self.groups > 1:
@@ -33,10 +35,12 @@ class RMSNorm(Part):
         self.weight: torch.Tensor | None = None
 
     def param_specs(self):
-        return {self.weight_name: ParamSpec((self.size,), "vector")}
+        return {self.weight_name: ParamSpec(() if self.scalar else (self.size,), "vector")}
 
     def load(self, tensors):
         self.weight = tensors[self.weight_name]
+        if self.scalar:
+            self.weight = self.weight.expand(self.size).contiguous()
         if self.weight_offset:
             self.weight = (self.weight.float() + self.weight_offset).contiguous()
 
@@ -58,6 +62,10 @@ class RMSNorm(Part):
         ``second``: another norm of the same size, groups and eps; the answer is then the pair
         ``(this norm's rows, the second norm's rows)`` of the same sum, made by one kernel."""
         n = stream.num_tokens if rows is None else (num_rows if num_rows is not None else rows.numel())
+        if stream.addends or stream.depth_weights is not None:
+            if self.center or self.groups > 1 or second is not None:
+                raise NotImplementedError("several outputs folded at once go with a plain rmsnorm")
+            return self._summed(stream, rows, n, normalise)
         if self.groups > 1 or second is not None or stream.pending_more is not None:
             if self.center:
                 raise NotImplementedError("layernorm: one norm of one pending output at a time")
@@ -98,6 +106,27 @@ class RMSNorm(Part):
             stream.add_vector = None
         return out
 
+
+    def _summed(self, stream: ResidualStream, rows, n: int, normalise: bool):
+        """Several outputs, some normed first, and the average over the depth if the stream has one."""
+        if stream.embed is not None or stream.pending is not None or stream.add_source or stream.add_vector is not None:
+            raise NotImplementedError("rmsnorm: a stream with addends holds nothing else that is pending")
+        keep = rows is None
+        depth = stream.depth_weights
+        out = torch.empty((n, self.size), dtype=self.ctx.dtype, device=self.ctx.device)
+        # the stream's first value is the first point, which stays: its average goes elsewhere
+        aliased = depth is not None and stream.resid.data_ptr() == stream.points.data_ptr()
+        target = (torch.empty_like(stream.resid) if aliased else stream.resid) if keep else None
+        self.ops.sum_norm(out, self.weight if normalise else None, self.eps, resid=stream.resid,
+                          items=[(a.value, a.norm_weight, a.norm_eps) for a in stream.addends], resid_out=target,
+                          points=stream.points, num_points=stream.num_points, depth_weights=depth, rows=rows, num_rows=n)
+        if keep:
+            stream.resid = target
+            stream.addends = []
+            if depth is not None:
+                stream.num_points += 1
+                stream.depth_weights = None
+        return out
 
     def _grouped(self, stream: ResidualStream, rows, n: int, normalise: bool, second):
         """The general kernel: groups, two pending outputs, two weights."""

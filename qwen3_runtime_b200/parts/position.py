@@ -126,6 +126,7 @@ class RotaryScaled(Part):
     ``kind="wavelength"`` (``factor, low, high, original``): with l = 2 pi / f, f stays where l < original / high,
     becomes f / factor where l > original / low, and in between, with s = (original / l - low) / (high - low),
     (1 - s) f / factor + s f (the schedule of Llama 3.1);
+    ``kind="linear"`` (``factor``): every f becomes f / factor;
     ``kind="ramp"`` (``factor, original, fast, slow``): with index(t) = rotary_dim ln(original / (2 pi t)) / (2 ln theta),
     lo = max(floor(index(fast)), 0), hi = min(ceil(index(slow)), rotary_dim - 1) and r_i = clamp((i - lo) /
     max(hi - lo, 0.001), 0, 1), f_i becomes f_i / factor * r_i + f_i * (1 - r_i), and cos and sin are multiplied
@@ -144,8 +145,8 @@ class RotaryScaled(Part):
             raise ValueError(f"rotary_dim={self.rotary_dim} must be a positive even number")
         if self.pairing not in ("half", "interleaved"):
             raise ValueError(f"rotation pairs are 'half' or 'interleaved', not {self.pairing!r}")
-        if self.scaling is not None and self.scaling.get("kind") not in ("wavelength", "ramp"):
-            raise ValueError(f"rotary_scaled: scaling kind is 'wavelength' or 'ramp', not {self.scaling.get('kind')!r}")
+        if self.scaling is not None and self.scaling.get("kind") not in ("wavelength", "ramp", "linear"):
+            raise ValueError(f"rotary_scaled: scaling kind is 'wavelength', 'ramp' or 'linear', not {self.scaling.get('kind')!r}")
         self.magnitude = 1.0
         if self.scaling is not None and self.scaling["kind"] == "ramp":
             self.magnitude = 0.1 * math.log(float(self.scaling["factor"])) + 1.0
@@ -157,6 +158,8 @@ class RotaryScaled(Part):
         sc = self.scaling
         if sc is None:
             return f
+        if sc["kind"] == "linear":
+            return [fi / float(sc["factor"]) for fi in f]
         factor, original = float(sc["factor"]), float(sc["original"])
         if sc["kind"] == "wavelength":
             low, high = float(sc["low"]), float(sc["high"])

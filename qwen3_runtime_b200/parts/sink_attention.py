@@ -13,7 +13,13 @@ back the pages that lie wholly between the kept first tokens and the window.  Fu
 the same kernel; without it positions do not enter the scores); ``softcap`` (scores become softcap *
 tanh(score / softcap) after the scale); ``values="keys"`` (there is no W_v: the values are the keys as
 projected, before norm and rotation); ``chunk`` (position i sees j <= i of its own chunk only, chunks of
-that many tokens counted from the sequence's first token).
+that many tokens counted from the sequence's first token); ``qkv_bias`` (biases ``q.b``, ``k.b``, ``v.b`` in the
+projections); ``own_kv=False`` (the layer has no key and value projections and reads the keys and values another
+layer has stored, under its own mask); ``value_turn`` (a rotary base: the value of position j is turned by j over
+all its dimensions before it is stored, pair m by ``j * base^(-2m / vdim)``, and a head's sum at position i is turned
+back by i).
+
+The part is a :class:`BranchMixer`: it runs alone or as a branch of the ``parallel`` mixer.
 """
 
 from __future__ import annotations
@@ -22,13 +28,11 @@ import torch
 
 from ..cache.layout import KVLayerSpec
 from ..config.spec import PartSpec
-from .base import BuildContext, ParamSpec, Part, StepContext, build_part, register_part
-from .linear_state import _pad_rows
+from .base import BuildContext, ParamSpec, StepContext, build_part, register_part
+from .linear_state import BranchMixer, _pad_rows
 
 
-class SinkWindowAttention(Part):
-    category = "mixer"
-
+class SinkWindowAttention(BranchMixer):
     def __init__(self, spec, ctx: BuildContext):
         super().__init__(spec, ctx)
         self.hidden_size = int(spec["hidden_size"])
@@ -64,7 +68,21 @@ class SinkWindowAttention(Part):
                                  "frequencies over at most the head's size; the position part offers otherwise")
         elif self.position.style != "none":
             raise ValueError(f"sink_window_attention has no {self.position.style!r} position encoding")
-        self.in_weight = self.o_weight = self.q_norm = self.k_norm = None
+        self.qkv_bias = bool(spec.get("qkv_bias", False))
+        self.own_kv = bool(spec.get("own_kv", True))
+        self.value_position = None
+        if spec.get("value_turn") is not None:
+            if self.vdim % 2 or self.values_are_keys:
+                raise ValueError("sink_window_attention: turned values have an even size and a projection of their own")
+            self.value_position = build_part("position", PartSpec("rotary_scaled", dict(
+                rotary_dim=self.vdim, theta=float(spec["value_turn"]),
+                pairing=getattr(self.position, "pairing", "half"))), ctx)
+        # q and k without norms: biases, rotations and the cache write are one kernel reading the step's turn tables
+        self.turned = self.qk_norm_eps is None and not self.values_are_keys
+        if not self.turned and (self.qkv_bias or not self.own_kv or self.value_position is not None):
+            raise ValueError("sink_window_attention: biases, shared keys and turned values go without q/k norms and with "
+                             "values of their own")
+        self.in_weight = self.o_weight = self.q_norm = self.k_norm = self.bias = None
         self._tables = None
         self.starts: list[int] = []
 
@@ -74,6 +92,10 @@ class SinkWindowAttention(Part):
                  "o": ParamSpec((W, H * Dv))}
         if self.values_are_keys:
             del specs["v"]
+        if not self.own_kv:
+            del specs["k"], specs["v"]
+        if self.qkv_bias:
+            specs.update({n + ".b": ParamSpec((specs[n].shape[0],), "vector") for n in ("q", "k", "v") if n in specs})
         if self.gate:
             specs["g"] = ParamSpec((H * Dv, W))
         if self.qk_norm_eps is not None:
@@ -85,12 +107,33 @@ class SinkWindowAttention(Part):
         if self.values_are_keys:  # no W_v: the value heads are read where the key heads are
             self.in_weight, starts = _pad_rows([tensors["q"], tensors["k"]] + ([tensors["g"]] if self.gate else []))
             self.starts = [starts[0], starts[1], starts[1], *starts[2:]]
+        elif not self.own_kv:
+            self.in_weight, starts = _pad_rows([tensors["q"]] + ([tensors["g"]] if self.gate else []))
+            self.starts = [0, 0, 0, *starts[1:]]
         else:
             blocks = [tensors["q"], tensors["k"], tensors["v"]] + ([tensors["g"]] if self.gate else [])
             self.in_weight, self.starts = _pad_rows(blocks)
+        if self.qkv_bias:
+            self.bias = torch.zeros(self.in_weight.shape[0], dtype=torch.float32, device=self.in_weight.device)
+            for name, at in zip(("q", "k", "v"), self.starts):
+                if name + ".b" in tensors:
+                    b = tensors[name + ".b"]
+                    self.bias[at:at + b.numel()] = b
         self.o_weight = tensors["o"].contiguous()
         self.q_norm = tensors.get("q.norm")
         self.k_norm = tensors.get("k.norm")
+
+    def input_weight(self):
+        return self.in_weight
+
+    def release_input_weight(self):
+        self.in_weight = None
+
+    def context_size(self):
+        return self.num_heads * self.vdim
+
+    def output_weight(self):
+        return self.o_weight
 
     def kernel_groups(self):
         groups = ["rope_kv", "attention_generic"]
@@ -148,13 +191,44 @@ class SinkWindowAttention(Part):
     def position_limit(self):
         return self.position.position_limit()
 
-    def forward(self, h: torch.Tensor, step: StepContext, cache) -> torch.Tensor:
+    def _turns(self, position, step: StepContext):
+        """The step's turn table for one set of frequencies, made by the first layer that asks for it."""
+        inv = position.inverse_frequencies()
+        key = ("turns", inv.data_ptr(), inv.numel())
+        if key not in step.extras:
+            step.extras[key] = self.ops.turn_table(step.positions, inv)
+        return step.extras[key]
+
+    def _turned_context(self, proj, step: StepContext, cache, ctx) -> None:
         ops = self.ops
         H, G, D, Dv = self.num_heads, self.num_kv_heads, self.dim, self.vdim
         s = self.starts
-        proj = ops.linear(h, self.in_weight)
         block_table = step.block_tables[cache.paged_index]
-        ctx = torch.empty((h.shape[0], H * Dv), dtype=h.dtype, device=h.device)
+        pairing = getattr(self.position, "pairing", "half")
+        qk_turns = self._turns(self.position, step) if self.position.style == "rotary" else None
+        v_turns = self._turns(self.value_position, step) if self.value_position is not None else None
+        gate = proj[:, s[3]:s[3] + H * Dv] if self.gate else None
+        ops.turn_store(proj, num_heads=H, num_kv_heads=G, head_dim=D, value_dim=Dv, k_start=s[1], v_start=s[2],
+                       bias=self.bias, qk_turns=qk_turns, value_turns=v_turns, positions=step.positions,
+                       token_seq=step.token_seq, block_table=block_table, k_pages=cache.k_pages, v_pages=cache.v_pages,
+                       page_size=cache.page_size, write_kv=cache.writes, pairing=pairing)
+        ops.paged_attention(proj, proj.stride(0), num_heads=H, num_kv_heads=G, head_dim=D, k_pages=cache.k_pages,
+                            v_pages=cache.v_pages, block_table=block_table, token_seq=step.token_seq,
+                            positions=step.positions, out=ctx, page_size=cache.page_size, scale=self.scale,
+                            window=self.window, step=step, value_dim=Dv, keep_first=self.keep_first, sink=self.sink,
+                            gate=gate, decode_slices=step.choices.get(self._slices_key()), chunk=self.chunk,
+                            softcap=self.softcap, value_turns=v_turns, pairing=pairing)
+
+    def context(self, proj, step: StepContext, cache, out, out_scale):
+        if out_scale != 1.0:
+            raise NotImplementedError("sink_window_attention: a branch's scale goes into the norm of its output")
+        ops = self.ops
+        if self.turned:
+            return self._turned_context(proj, step, cache, out)
+        H, G, D, Dv = self.num_heads, self.num_kv_heads, self.dim, self.vdim
+        s = self.starts
+        ctx = out
+        block_table = step.block_tables[cache.paged_index]
         gate = proj[:, s[3]:s[3] + H * Dv] if self.gate else None
         fusable = getattr(ops, "decode_new_token_ok", None)
         rotary = self.position.style == "rotary"
@@ -183,7 +257,7 @@ class SinkWindowAttention(Part):
                                values_are_keys=self.values_are_keys),
                 num_splits=step.choices.get(self._slices_key()), longest=step.kv_longest, step=step,
                 keep_first=self.keep_first, sink=self.sink, gate=gate, softcap=self.softcap)
-            return ops.linear(ctx, self.o_weight)
+            return
         ops.qk_norm_store(proj, num_heads=H, num_kv_heads=G, head_dim=D, value_dim=Dv, k_start=s[1], v_start=s[2],
                           q_weight=self.q_norm, k_weight=self.k_norm,
                           eps=self.qk_norm_eps if self.qk_norm_eps is not None else 0.0, positions=step.positions,
@@ -197,7 +271,6 @@ class SinkWindowAttention(Part):
                             window=self.window, step=step, value_dim=Dv, keep_first=self.keep_first, sink=self.sink,
                             gate=gate, decode_slices=step.choices.get(self._slices_key()),
                             **(dict(chunk=self.chunk, softcap=self.softcap) if self.chunk or self.softcap else {}))
-        return ops.linear(ctx, self.o_weight)
 
 
 register_part("mixer", "sink_window_attention", SinkWindowAttention)

@@ -88,6 +88,134 @@ class TorchOps:
             out2[:n] = (unit * weight2.float()).to(out2.dtype)
         return out
 
+    def sum_norm(self, out, weight, eps, *, resid, items, resid_out=None, points=None, num_points=0, depth_weights=None,
+                 rows=None, num_rows=None):
+        n = out.shape[0] if num_rows is None else num_rows
+        src = rows[:n].long() if rows is not None else torch.arange(n, device=out.device)
+        v = resid[src].float()
+        for value, w, e in items:
+            if value.dim() == 3:
+                x = value[0][src]
+                for p in range(1, value.shape[0]):
+                    x = x + value[p][src]
+            else:
+                x = value[src].float()
+            if w is not None:
+                x = (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + e)) * w.float()
+            v = v + x
+        if depth_weights is not None:
+            if resid_out is not None:
+                points[num_points, src] = v
+            acc = torch.zeros_like(v)
+            for j in range(num_points):
+                acc = acc + depth_weights[j] * points[j, src]
+            v = acc + depth_weights[num_points] * v
+        if resid_out is not None:
+            resid_out[src] = v
+        if weight is None:
+            out[:n] = v.to(out.dtype)
+        else:
+            out[:n] = ((v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)) * weight.float()).to(out.dtype)
+        return out
+
+    def embed_norm(self, ids, table, weight, eps, out):
+        x = table[ids[: out.shape[0]].long()].float()
+        out.copy_((x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)) * weight.float())
+        return out
+
+    def turn_table(self, positions, inv_freq):
+        ang = positions.float()[:, None] * inv_freq.float()[None, :]
+        return torch.stack([ang.cos(), ang.sin()], dim=1).contiguous()
+
+    @staticmethod
+    def _turn_by(x, turns, pairing, direction=1.0):
+        """x [T, heads, n] float: the leading 2 * pairs elements turn by the table's angles (or back)."""
+        if turns is None:
+            return x
+        pairs = turns.shape[2]
+        c, s = turns[:, 0][:, None, :], turns[:, 1][:, None, :] * direction
+        out = x.clone()
+        if pairing == "interleaved":
+            u, v = x[..., 0:2 * pairs:2], x[..., 1:2 * pairs:2]
+            out[..., 0:2 * pairs:2], out[..., 1:2 * pairs:2] = u * c - v * s, v * c + u * s
+        else:
+            u, v = x[..., :pairs], x[..., pairs:2 * pairs]
+            out[..., :pairs], out[..., pairs:2 * pairs] = u * c - v * s, v * c + u * s
+        return out
+
+    def turn_store(self, proj, *, num_heads, num_kv_heads, head_dim, value_dim, k_start, v_start, bias, qk_turns,
+                   value_turns, positions, token_seq, block_table, k_pages, v_pages, page_size, write_kv,
+                   pairing="half"):
+        T = proj.shape[0]
+        H, G, D, Dv = num_heads, num_kv_heads, head_dim, value_dim
+        x = proj.float()
+        if bias is not None:
+            x = x + bias.float()[: proj.shape[1]]
+        q = self._turn_by(x[:, : H * D].reshape(T, H, D), qk_turns, pairing)
+        proj[:, : H * D] = q.reshape(T, H * D).to(proj.dtype)
+        if not write_kv:
+            return
+        k = self._turn_by(x[:, k_start:k_start + G * D].reshape(T, G, D), qk_turns, pairing).to(proj.dtype)
+        v = self._turn_by(x[:, v_start:v_start + G * Dv].reshape(T, G, Dv), value_turns, pairing).to(proj.dtype)
+        for t in range(T):
+            p = int(positions[t])
+            page = int(block_table[int(token_seq[t]), p // page_size])
+            if page < 0:
+                continue
+            k_pages[page, :, p % page_size, :] = k[t]
+            v_pages[page, :, p % page_size, :] = v[t]
+
+    # ---- gated delta rule ----------------------------------------------------------------
+    def delta_rule(self, x, z, b, *, heads, kv_heads, dim, value_dim, conv_weight, ring, dt_bias, neg_a, state, positions,
+                   token_seq, cu_seqlens, state_slots, num_seqs, q_scale):
+        T, H, G, D, Dv = x.shape[0], heads, kv_heads, dim, value_dim
+        taps = conv_weight.shape[0]
+        u = x.float()
+        y = torch.zeros_like(u)
+        for s in range(num_seqs):
+            slot = int(state_slots[s])
+            t0, t1 = int(cu_seqlens[s]), int(cu_seqlens[s + 1])
+            for t in range(t0, t1):
+                p = int(positions[t])
+                for j in range(taps):
+                    back = taps - 1 - j
+                    if p - back >= 0:
+                        y[t] += conv_weight[j] * (u[t - back] if t - back >= t0 else ring[slot, (p - back) % taps])
+            if taps > 1:
+                for t in range(max(t0, t1 - taps), t1):
+                    ring[slot, int(positions[t]) % taps] = u[t]
+        y = y / (1 + torch.exp(-y))
+        q, k = y[:, : G * D].reshape(T, G, D), y[:, G * D:2 * G * D].reshape(T, G, D)
+        v = y[:, 2 * G * D:].to(x.dtype).float().reshape(T, H, Dv)
+        q = (q * torch.rsqrt(q.pow(2).sum(-1, keepdim=True) + 1e-6) * q_scale).repeat_interleave(H // G, dim=1)
+        k = (k * torch.rsqrt(k.pow(2).sum(-1, keepdim=True) + 1e-6)).repeat_interleave(H // G, dim=1)
+        g = torch.exp(neg_a[None, :, None] * torch.nn.functional.softplus(z.reshape(T, H, D) + dt_bias.reshape(H, D),
+                                                                          threshold=60.0))
+        beta = torch.sigmoid(b.float())
+        out = torch.empty((T, H, Dv), dtype=torch.float32, device=x.device)
+        for s in range(num_seqs):
+            slot = int(state_slots[s])
+            S = state[slot].clone()
+            for t in range(int(cu_seqlens[s]), int(cu_seqlens[s + 1])):
+                S = g[t][:, :, None] * S
+                w = beta[t][:, None] * (v[t] - torch.einsum("hdv,hd->hv", S, k[t]))
+                S = S + k[t][:, :, None] * w[:, None, :]
+                out[t] = torch.einsum("hdv,hd->hv", S, q[t])
+            state[slot] = S
+        return out
+
+    def delta_step_ok(self, dim, value_dim):
+        return True
+
+    def delta_step(self, x, low_a, low_g, b, out, *, a2, g2, norm_weight, eps, **kw):
+        T, H, Dv = x.shape[0], kw["heads"], kw["value_dim"]
+        z = (low_a.float() @ a2.float().t())
+        o = self.delta_rule(x, z, b, token_seq=None, **kw)
+        gate = torch.sigmoid(low_g.float() @ g2.float().t()).reshape(T, H, Dv)
+        o = (o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)) * norm_weight.float() * gate
+        out.copy_(o.reshape(T, H * Dv).to(out.dtype))
+        return out
+
     def bigram_embed(self, ids, *, embed, scale, bigram, buckets, mul_prev, mul_cur, prev_state, positions,
                      token_seq, cu_seqlens, state_slots, num_seqs, out, copy=None):
         T = out.shape[0]
@@ -357,7 +485,8 @@ class TorchOps:
     # ---- attention --------------------------------------------------------------------
     def paged_attention(self, q, q_stride, *, num_heads, num_kv_heads, head_dim, k_pages, v_pages, block_table,
                         token_seq, positions, out, page_size, scale, window, step=None, decode_slices=None,
-                        value_dim=None, keep_first=0, sink=None, gate=None, chunk=None, softcap=None):
+                        value_dim=None, keep_first=0, sink=None, gate=None, chunk=None, softcap=None, value_turns=None,
+                        pairing="half"):
         T = out.shape[0]
         D = head_dim
         group = num_heads // num_kv_heads
@@ -383,7 +512,10 @@ class TorchOps:
                 probs = torch.softmax(scores, dim=-1)[:, :-1]
             else:
                 probs = torch.softmax(scores, dim=-1)
-            res = torch.einsum("hn,nhd->hd", probs, vh).reshape(-1)
+            res = torch.einsum("hn,nhd->hd", probs, vh)
+            if value_turns is not None:  # turned back by the token's angles
+                res = self._turn_by(res[None], value_turns[t:t + 1], pairing, direction=-1.0)[0]
+            res = res.reshape(-1)
             if gate is not None:
                 res = res * torch.sigmoid(gate[t].float())
             out[t] = res.to(out.dtype)
