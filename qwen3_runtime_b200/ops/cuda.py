@@ -119,6 +119,27 @@ _SIGNATURES = {
         "q3_qk_norm_store": [c_int, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
                              c_void_p, c_float, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p,
                              c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+        "q3_turn_table": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p],
+        "q3_turn_store": [c_int, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
+                          c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
+                          c_int, c_void_p],
+    },
+    "depth_norm": {
+        "q3_sum_norm": [c_int, c_int, *([c_void_p, c_int, c_long, c_void_p, c_float] * 4), c_void_p, c_void_p, c_void_p,
+                        c_long, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p],
+        "q3_embed_norm": [c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p],
+    },
+    "delta_state": {
+        "q3_delta_prepare": [c_int, c_void_p, c_long, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                             c_void_p, c_void_p, c_void_p, c_void_p, c_long, c_float, c_void_p, c_void_p, c_void_p,
+                             c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
+        "q3_ring_update": [c_int, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                           c_void_p],
+        "q3_delta_scan": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                          c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
+        "q3_delta_step": [c_int, c_void_p, c_long, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                          c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p,
+                          c_void_p, c_float, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_void_p],
     },
     "attention_generic": {
         "q3_paged_attention_generic": [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,

@@ -135,6 +135,7 @@ class DecoderModel:
         """Run the step's tokens through every run entry; float32 logits ``[R, V]`` at
         ``step.logit_rows`` (None when no logits are wanted)."""
         s = self.spec
+        step.extras = {}  # a captured step runs twice (warm-up, capture): nothing made by the first run is reused
         if self.embedding is not None:
             stream = self.embedding.start(step, storage.view(EMBEDDING_CACHE), keep_source=self.keeps_source,
                                           num_points=self.num_points)

@@ -77,6 +77,8 @@ def turned_values_core(q, k, v, scale, chunk, base):
 
 
 def _qk_freqs(rot, dtype):
+    if rot is None:
+        return torch.zeros(0, dtype=dtype)
     factor = float((rot.get("scaling") or {}).get("factor", 1.0))
     return frequencies(rot["dims"], rot["base"], dtype, factor)
 
@@ -91,7 +93,7 @@ def biased_attention(h, t, p, m, kept):
     T = h.shape[0]
     H, G, D, Dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
     pos = torch.arange(T)
-    freqs = _qk_freqs(m["rot"], h.dtype)
+    freqs = _qk_freqs(m.get("rot"), h.dtype)
     q = _r(rotate(_r(h @ t[p + "q"].T + t[p + "q.b"]).view(T, H, D), pos, freqs))
     if kept is None:
         k = _r(rotate(_r(h @ t[p + "k"].T + t[p + "k.b"]).view(T, G, D), pos, freqs))
