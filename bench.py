@@ -55,6 +55,10 @@ kinds and a roofline fraction per kind):
                    sink and an output gate, layer norms on the sublayers' outputs only, a layer that runs another
                    layer's weights) at two layer sizes beside the Logesun design at equal sizes, its closest
                    relative (dense feed-forwards in both);
+* ``pevazen``      the Pevazen design (attention under a chunked mask with turned values beside the gated delta
+                   rule, attention with biases and with another layer's keys, one norm per layer, averages over
+                   the depth) at two layer sizes beside the Puladra design at equal sizes, its closest relative
+                   (windowed attention beside retention, gated linear attention);
 * ``decode``, ``latency``, ``batch8``, ``throughput``, ``prefill``, ``longctx``: the six closed
                    batches of the reference's own harness (bench/workloads.py:34-43) at Qwen3-4B
                    sizes, with its token budget rule (bench/workloads.py:52-64).
@@ -67,6 +71,7 @@ timed iterations.  ``--impl reference`` runs the unmodified reference installed 
 from __future__ import annotations
 
 import argparse
+import dataclasses
 import json
 import os
 import statistics
@@ -105,7 +110,7 @@ BASELINE_TOK_S = 693.26
 # (concurrency = requests, prompt tokens, output tokens) of the reference's closed batches
 CLOSED_CASES = {"decode": (1, 256, 512), "latency": (1, 512, 128), "batch8": (8, 256, 128),
                 "throughput": (16, 256, 128), "prefill": (1, 2048, 16), "longctx": (1, 8192, 64)}
-WORKLOADS = ("default", "decode512", "batch48", "32b", "logesun", "puladra", "medilix", "tabisun", *CLOSED_CASES)
+WORKLOADS = ("default", "decode512", "batch48", "32b", "logesun", "puladra", "medilix", "tabisun", "pevazen", *CLOSED_CASES)
 
 # Layer sizes for the Puladra design that resemble real models of its kinds of layer: gated linear
 # attention with keys of half and values of the full width, windowed attention with grouped key/value
@@ -151,6 +156,19 @@ TABISUN_SIZES = {
     "w4096": dict(width=4096, ff=12288, vocab=32000, layers=4, chunk=2048,
                   diff=dict(heads=32, kv_heads=8, dim=64, vdim=128), kv=dict(heads=32, kv_heads=8, dim=128, rot=64),
                   latent=dict(heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512)),
+}
+
+# Layer sizes for the Pevazen design: attention with grouped heads of 128 under chunks of 2,048 tokens (half of each
+# head rotated, biases; beside the delta rule with turned values and the whole head rotated), the gated delta rule with
+# keys and values of 128 and a convolution of four taps, dense SwiGLU feed-forwards.  Four layers (parallel,
+# attention, parallel, attention on the second one's keys).  Beside each runs Puladra (parallel, gla, parallel, gla)
+# with the same attention, state sizes and convolution, a window of the chunk's size, and routed experts whose active
+# width is the dense feed-forward's.
+PEVAZEN_SIZES = {
+    "w2048": dict(width=2048, ff=8192, vocab=32000, layers=4, chunk=2048, att=dict(heads=16, kv_heads=4, dim=128, rot=64),
+                  delta=dict(heads=16, kv_heads=8, dim=128, vdim=128, conv=4, rank=64), experts=16, top=4),
+    "w4096": dict(width=4096, ff=12288, vocab=32000, layers=4, chunk=2048, att=dict(heads=32, kv_heads=8, dim=128, rot=64),
+                  delta=dict(heads=32, kv_heads=16, dim=128, vdim=128, conv=4, rank=128), experts=16, top=4),
 }
 
 # Layer sizes for the Logesun design (attention through a latent with a window and a sink, routed
@@ -736,6 +754,54 @@ def run_tabisun(args, pk) -> dict:
                                    twin=("logesun", _logesun_twin_config, "the Logesun design"))
 
 
+def _pevazen_config(z: dict):
+    from qwen3_runtime_b200.config import PevazenConfig
+    from qwen3_runtime_b200.config.pevazen_config import (ChunkedAttentionConfig, DeltaConfig, PevazenLayerConfig,
+                                                          SideBySideConfig)
+    from qwen3_runtime_b200.config.tabisun_config import RotaryConfig
+
+    a, d = z["att"], z["delta"]
+    att = ChunkedAttentionConfig(heads=a["heads"], kv_heads=a["kv_heads"], dim=a["dim"], vdim=a["dim"],
+                                 scale=a["dim"] ** -0.5, chunk=z["chunk"], rot=RotaryConfig(dims=a["rot"], base=1e4))
+    side = SideBySideConfig(
+        left=dataclasses.replace(att, rot=RotaryConfig(dims=a["dim"], base=5e5, scaling=(("factor", 4.0),))),
+        right=DeltaConfig(heads=d["heads"], kv_heads=d["kv_heads"], dim=d["dim"], vdim=d["vdim"], conv=d["conv"],
+                          decay_rank=d["rank"], gate_rank=d["rank"]))
+    layers = (PevazenLayerConfig("parallel", side, z["ff"]), PevazenLayerConfig("attention", att, z["ff"]),
+              PevazenLayerConfig("parallel", side, z["ff"]),
+              PevazenLayerConfig("attention", dataclasses.replace(att, kv_from=1), z["ff"]))
+    return PevazenConfig(vocab=z["vocab"], width=z["width"], norm_eps=1e-6, layers=layers)
+
+
+def _puladra_beside_pevazen_config(z: dict):
+    """Puladra at the sizes of a Pevazen entry: its windowed attention has the chunked attention's heads and sizes (the
+    window is the chunk's size), retention and gated linear attention have the delta rule's states, the routed experts'
+    active width is the dense feed-forward's; no shared expert, no token input."""
+    from qwen3_runtime_b200.config import PuladraConfig
+    from qwen3_runtime_b200.config.puladra_config import (GlaConfig, MoeConfig, ParallelConfig, PuladraLayerConfig,
+                                                          RetentionConfig, RotationConfig, WindowAttentionConfig)
+
+    a, d = z["att"], z["delta"]
+    gla = GlaConfig(heads=d["heads"], dim=d["dim"], vdim=d["vdim"], tau=16.0, decay_rank=d["rank"])
+    par = ParallelConfig(
+        left=WindowAttentionConfig(heads=a["heads"], kv_heads=a["kv_heads"], dim=a["dim"], vdim=a["dim"],
+                                   scale=a["dim"] ** -0.5, conv=d["conv"], rot=RotationConfig(a["dim"], 10000.0),
+                                   window=z["chunk"]),
+        right=RetentionConfig(heads=d["heads"], dim=d["dim"], vdim=d["vdim"],
+                              decay=tuple(1.0 - 2.0 ** (-5 - (i % 8)) for i in range(d["heads"])),
+                              rot=RotationConfig(d["dim"], 10000.0)),
+        left_scale=1.0, right_scale=1.0)
+    moe = MoeConfig(experts=z["experts"], top=z["top"], ff=z["ff"] // z["top"], shared_ff=0)
+    layers = tuple(PuladraLayerConfig("parallel", par, moe) if i % 2 == 0 else PuladraLayerConfig("gla", gla, moe)
+                   for i in range(z["layers"]))
+    return PuladraConfig(vocab=z["vocab"], width=z["width"], norm_eps=1e-6, layers=layers, logit_scale=1.0, side_dim=0)
+
+
+def run_pevazen(args, pk) -> dict:
+    return run_design_beside_dense(args, pk, "pevazen", "Pevazen", PEVAZEN_SIZES, _pevazen_config,
+                                   twin=("puladra", _puladra_beside_pevazen_config, "the Puladra design"))
+
+
 def _puladra_twin_config(z: dict):
     """Puladra at the sizes of a Medilix entry: its gated linear attention has the mlstm's heads and sizes, its
     windowed attention the attention's, its retention the wkv's."""
@@ -835,6 +901,8 @@ def run_workload_ours(args) -> dict:
         return run_medilix(args, pk)
     if args.workload == "tabisun":
         return run_tabisun(args, pk)
+    if args.workload == "pevazen":
+        return run_pevazen(args, pk)
     cases = workload_prompts(args.workload, np)
     results, cfg, build_s, engine = {}, None, 0.0, None
     clocks = ClockSampler()
@@ -1092,7 +1160,7 @@ def main() -> int:
     args.warmup = max(3, args.warmup)
     if args.workload == "default":
         result = run_reference(args) if args.impl == "reference" else run_ours(args)
-    elif args.workload in ("logesun", "puladra", "medilix", "tabisun") and args.impl == "reference":
+    elif args.workload in ("logesun", "puladra", "medilix", "tabisun", "pevazen") and args.impl == "reference":
         result = {"impl": "reference", "workload": args.workload,
                   "unavailable": "the reference has no model of this design (it serves Qwen3 dense only)"}
     else:

@@ -1,8 +1,8 @@
 // Causal attention of prompt portions over the paged cache on the 5th-generation tensor
 // cores: S = Q K^T and O += P V are tcgen05.mma with accumulators in tensor memory, Q, K and V
 // tiles arrive by TMA (128-byte swizzle) straight from the QKV buffer and the cache pages.
-// bfloat16, head_dim 128, group size a divisor of 128, page size 8/16/32/64, no window; the
-// mma.sync kernel of attention_prefill.cu serves everything else.
+// bfloat16, head_dim 128, group size a divisor of 128, page size 8/16/32/64, no window (a chunked mask
+// and turned values are options); the mma.sync kernels serve everything else.
 //
 // Work item: (sequence, kv head, two consecutive blocks of 128 rows, A and B); rows are the
 // (query token, head of the group) pairs in token-major order, so one 3-D TMA box
@@ -67,7 +67,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
                             const __grid_constant__ CUtensorMap tmap_v, const int* __restrict__ block_table,
                             int max_pages, const int* __restrict__ kv_lens, const int* __restrict__ cu_seqlens,
                             bf16* __restrict__ out, int num_seqs, int num_work, int nq, int nkv, int ps,
-                            float scale_log2, int skip_single, int* __restrict__ error_word) {
+                            float scale_log2, int skip_single, int chunk, const float* __restrict__ turns,
+                            int* __restrict__ error_word) {
   extern __shared__ unsigned char smem_raw[];
   unsigned char* base = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   unsigned char* q_s = base;                         // 2 blocks x [2 halves][128 rows][128 B]
@@ -138,13 +139,17 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
     const int base_pos = kv_len - q_len;
     // row blocks A and B of this item; B may not exist (odd number of blocks)
     int row0[2], p_max[2], tiles[2];
+    // under a chunked mask the item's first visible key is that of its first row; tiles count from the tile it is in
+    const int p_first = base_pos + 2 * s_item[1] * BLOCK_M / G;
+    const int k_lo = chunk > 0 ? p_first / chunk * chunk : 0;
+    const int tile0 = k_lo / BLOCK_N;
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
       row0[x] = (2 * s_item[1] + x) * BLOCK_M;
       const bool live = row0[x] < rows;
       const int last_row = min(rows, row0[x] + BLOCK_M) - 1;
       p_max[x] = live ? base_pos + last_row / G : -1;
-      tiles[x] = live ? p_max[x] / BLOCK_N + 1 : 0;
+      tiles[x] = live ? p_max[x] / BLOCK_N + 1 - tile0 : 0;
     }
     const int num_tiles = max(tiles[0], tiles[1]);  // B lies after A, so this is B's count when B exists
     const int p_last = max(p_max[0], p_max[1]);
@@ -171,8 +176,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
         // pages of this tile that exist in the block table (the rest of the tile is masked)
         int page = -1;
         if (my_page < pages_per_tile) {
-          const int pi = j * pages_per_tile + my_page;
-          if (pi < max_pages && pi * ps <= p_last) page = bt[pi];
+          const int pi = (tile0 + j) * pages_per_tile + my_page;
+          if (pi < max_pages && pi * ps <= p_last && (pi + 1) * ps > k_lo) page = bt[pi];
         }
         const uint32_t boxes = __popc(__ballot_sync(0xffffffffu, page >= 0));
         const uint32_t bytes = boxes * (uint32_t)ps * 128u;
@@ -260,6 +265,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
       const int R = row0[x] + r;
       const bool row_ok = R < rows;
       const int pos = row_ok ? base_pos + R / G : -1;
+      const int lo = chunk > 0 && row_ok ? pos / chunk * chunk : 0;  // the row's first visible key
       const int my_tiles = tiles[x];
       const uint32_t lane_base = tmem + x * TMEM_BLOCK + ((uint32_t)(quarter * 32) << 16);
       const uint32_t o_addr = lane_base + 2 * BLOCK_N;
@@ -280,13 +286,20 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
         tmem_load32(lane_base + st * BLOCK_N, sa);
         tmem_load32(lane_base + st * BLOCK_N + 32, sb);
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-        const int key0 = j * BLOCK_N;
+        const int key0 = (tile0 + j) * BLOCK_N;
         float mx = -INFINITY;
         if (key0 + BLOCK_N - 1 > pos) {  // the tile crosses this row's diagonal
 #pragma unroll
           for (int c = 0; c < 32; ++c) {
             if (key0 + c > pos) sa[c] = 0xff800000u;       // -inf
             if (key0 + 32 + c > pos) sb[c] = 0xff800000u;
+          }
+        }
+        if (key0 < lo) {  // keys of an earlier chunk
+#pragma unroll
+          for (int c = 0; c < 32; ++c) {
+            if (key0 + c < lo) sa[c] = 0xff800000u;
+            if (key0 + 32 + c < lo) sb[c] = 0xff800000u;
           }
         }
         {  // eight independent running maxima: a single chain of 64 would expose its latency
@@ -360,14 +373,14 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
             asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
           }
         }
-        // keys of this tile past the item's last position hold whatever the page held: zero their
-        // value rows before PV reads them (both blocks do, each before its own PV; keys between the
-        // blocks' last positions are real and only masked)
-        if (key0 + BLOCK_N - 1 > p_last) {
+        // keys of this tile past the item's last position hold whatever the page held, keys before its first
+        // visible one may not have been loaded at all: zero their value rows before PV reads them (both blocks
+        // do, each before its own PV; keys between the blocks' last positions are real and only masked)
+        if (key0 + BLOCK_N - 1 > p_last || key0 < k_lo) {
           ok = mbar_wait(bar(BAR_V_FULL + vst), (j / KV_STAGES) & 1, &abort_flag);
           if (!ok) break;
           const int vrow = r & 63, half = r >> 6;
-          if (key0 + vrow > p_last) {
+          if (key0 + vrow > p_last || key0 + vrow < k_lo) {
             uint4* dst = reinterpret_cast<uint4*>(v_s + vst * KV_BYTES + half * (KV_BYTES / 2) + vrow * 128);
 #pragma unroll
             for (int ch = 0; ch < 8; ++ch) dst[ch] = make_uint4(0, 0, 0, 0);
@@ -382,8 +395,34 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         const float inv = 1.f / l_run;
         bf16* dst = row_ok ? out + ((long)(tok0 + R / G) * nq + kvh * G + R % G) * D : nullptr;
+        if (turns) {  // turned values: the sum is turned back, element c with element c + D / 2
+          const float* cs = row_ok ? turns + (long)(tok0 + R / G) * D : nullptr;  // cos (D / 2), sin (D / 2)
 #pragma unroll 1
-        for (int c0 = 0; c0 < D; c0 += 32) {
+          for (int c0 = 0; c0 < D / 2; c0 += 32) {
+            uint32_t ua[32], ub[32];
+            tmem_load32(o_addr + c0, ua);
+            tmem_load32(o_addr + D / 2 + c0, ub);
+            asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+            if (row_ok) {
+#pragma unroll
+              for (int c = 0; c < 32; c += 8) {
+                float co[8], sn[8], x8[8], y8[8];
+                load8(cs + c0 + c, co);
+                load8(cs + D / 2 + c0 + c, sn);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) {
+                  const float u = __uint_as_float(ua[c + e]) * inv, v = __uint_as_float(ub[c + e]) * inv;
+                  x8[e] = u * co[e] + v * sn[e];
+                  y8[e] = v * co[e] - u * sn[e];
+                }
+                store8(dst + c0 + c, x8);
+                store8(dst + D / 2 + c0 + c, y8);
+              }
+            }
+          }
+        }
+#pragma unroll 1
+        for (int c0 = 0; c0 < D && !turns; c0 += 32) {
           uint32_t ov[32];
           tmem_load32(o_addr + c0, ov);
           asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -416,12 +455,16 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
 // h * 128.  kpages / vpages: [num_rows_kv / (nkv * ps), nkv, ps, 128] bf16 of one layer, num_rows_kv
 // rows of 128 in all.  num_work = sum over served sequences of ceil(ceil(q_len * (nq / nkv) / 128) / 2).
 // Returns Q3_ERR_UNSUPPORTED for shapes this kernel does not take (the caller then uses the
-// mma.sync kernel).  error_word: device int set to 2 if a wait inside the kernel expired.
+// mma.sync kernel).  chunk > 0: a token sees the keys of its own chunk of that many tokens only.  turns: null, or
+// fp32 [num_tokens, 2, 64], cos then sin per pair (m, m + 64): the cached values are turned by their positions and a
+// head's result is turned back by its token's angles.  error_word: device int set to 2 if a wait inside the kernel expired.
 Q3_EXPORT int q3_paged_attention_prefill_tc(const void* q, int q_stride, int num_tokens, const void* kpages,
                                             const void* vpages, long num_rows_kv, const int* block_table,
                                             int max_pages, const int* kv_lens, const int* cu_seqlens, void* out,
                                             int num_seqs, int num_work, int nq, int nkv, int head_dim, int ps,
-                                            float scale, int skip_single, int* error_word, cudaStream_t stream) {
+                                            float scale, int skip_single, int chunk, const float* turns,
+                                            int* error_word, cudaStream_t stream) {
+  if (chunk < 0 || ((uintptr_t)turns & 15)) return Q3_ERR_ARGUMENT;
   if (!q || !kpages || !vpages || !block_table || !kv_lens || !cu_seqlens || !out) return Q3_ERR_ARGUMENT;
   if (nq < 1 || nkv < 1 || nq % nkv) return Q3_ERR_ARGUMENT;
   const int G = nq / nkv;
@@ -458,6 +501,6 @@ Q3_EXPORT int q3_paged_attention_prefill_tc(const void* q, int q_stride, int num
   prefill_attention_tc_kernel<<<grid, THREADS, SMEM_BYTES, stream>>>(tq, tk, tv, block_table, max_pages, kv_lens,
                                                                     cu_seqlens, (bf16*)out, num_seqs, num_work, nq,
                                                                     nkv, ps, scale * 1.4426950408889634f,
-                                                                    skip_single, error_word);
+                                                                    skip_single, chunk, turns, error_word);
   return q3_launch_status();
 }

@@ -203,7 +203,15 @@ _SIGNATURES = {
     "attention_prefill_tc": {
         "q3_paged_attention_prefill_tc": [c_void_p, c_int, c_int, c_void_p, c_void_p, ctypes.c_long, c_void_p, c_int,
                                           c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                                          c_float, c_int, c_void_p, c_void_p],
+                                          c_float, c_int, c_int, c_void_p, c_void_p, c_void_p],
+    },
+    "attention_chunk": {
+        "q3_chunk_attention_prefill": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
+                                       c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int,
+                                       c_int, c_void_p, c_int, c_int, c_void_p],
+        "q3_chunk_attention_decode": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+                                      c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
+                                      c_int, c_float, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
     },
     "gemm_f32": {
         "q3_gemm_f32": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
@@ -275,6 +283,7 @@ class CudaOps:
         self.fuse_decode_new_token = True   # False: always the separate q/k norm + rotation + store kernel
         self.latent_attention_tc = True     # False: attention over latent rows always on the general kernel
         self.experts_tc = True              # False: the experts' products always on the FMA kernels
+        self.chunk_tc = True                # False: attention under chunks or with turned values on the general kernel
         self.differential_tc = True         # False: differential attention always on the general kernel
         self._tickets: torch.Tensor | None = None
         self._argmax_tickets: torch.Tensor | None = None
@@ -1258,8 +1267,8 @@ class CudaOps:
                     _ptr(q), q_stride, q.shape[0], _ptr(k_pages), _ptr(v_pages),
                     k_pages.shape[0] * num_kv_heads * page_size, _ptr(block_table), block_table.shape[1],
                     _ptr(step.kv_lens), _ptr(step.cu_seqlens), _ptr(out), step.num_seqs, pairs, num_heads,
-                    num_kv_heads, head_dim, page_size, float(scale), 1, _ptr(self._error_word(out.device)),
-                    self._stream())
+                    num_kv_heads, head_dim, page_size, float(scale), 1, 0, None,
+                    _ptr(self._error_word(out.device)), self._stream())
                 if self.timing is not None:
                     self._costs(*self._attention_cost(step, num_heads, num_kv_heads, head_dim, out, prompts=True))
                     with self._timed("paged_attention_prefill_tc"):
@@ -1290,6 +1299,11 @@ class CudaOps:
                     num_splits=self.decode_slices_for(singles, num_kv_heads, head_dim,
                                                       window + keep_first if window else window), **extras)
             return out
+        if (self.chunk_tc and step is not None and out.dtype == torch.bfloat16 and plain and not window and not softcap
+                and head_dim % 8 == 0 and Dv % 8 == 0 and num_heads // num_kv_heads <= 16 and q_stride % 8 == 0
+                and out.stride(0) % 2 == 0 and q.data_ptr() % 16 == 0 and out.data_ptr() % 4 == 0):
+            return self._chunk_attention(q, q_stride, num_heads, num_kv_heads, head_dim, Dv, k_pages, v_pages, block_table,
+                                         out, page_size, scale, chunk, step, value_turns, pairing)
         if self.timing is not None and step is not None:
             self._costs(*self._attention_cost(step, num_heads, num_kv_heads, head_dim, out))
         self._call("attention_generic", "q3_paged_attention_generic", "paged_attention",
@@ -1300,6 +1314,96 @@ class CudaOps:
                   chunk, softcap, _ptr(value_turns), value_turns.shape[2] if value_turns is not None else 0,
                   self.PAIRINGS[pairing])
         return out
+
+    def _chunk_attention(self, q, q_stride, H, G, D, Dv, k_pages, v_pages, block_table, out, page_size, scale, chunk, step,
+                         turns, pairing):
+        """:meth:`paged_attention` in bfloat16 with keys and values of sizes of their own, under a chunked mask
+        (``chunk`` 0: none), values possibly turned: prompt portions on the tensor cores (tcgen05 where heads of 128 and
+        the page size allow it, csrc/attention_prefill_tc.cu, else csrc/attention_chunk.cu), one-token sequences in
+        slices of their visible keys (csrc/attention_chunk.cu)."""
+        group = H // G
+        pairs = turns.shape[2] if turns is not None else 0
+        singles = step.num_seqs if step.decode_only else step.num_single
+        cost = (lambda prompts: self._costs(*self._chunk_cost(step, H, G, D, Dv, chunk, out, prompts))) \
+            if self.timing is not None else None
+        if not step.decode_only:
+            cu = step.host_cu_seqlens
+            skip = int(singles > 0)
+            qlens = [cu[b + 1] - cu[b] for b in range(step.num_seqs)]
+            served = [n for n in qlens if n > skip]
+            done = not served
+            if (served and D == 128 and Dv == 128 and 128 % group == 0 and page_size in (8, 16, 32, 64)
+                    and out.stride(0) == H * Dv and self.prefill_attention == "tcgen05"
+                    and (turns is None or (pairs == 64 and pairing == "half"))):
+                work = sum(-(-(-(-n * group // 128)) // 2) for n in served)  # two row blocks per work item
+                self.launches += 1
+                launch = lambda: self._get("attention_prefill_tc", "q3_paged_attention_prefill_tc")(  # noqa: E731
+                    _ptr(q), q_stride, q.shape[0], _ptr(k_pages), _ptr(v_pages), k_pages.shape[0] * G * page_size,
+                    _ptr(block_table), block_table.shape[1], _ptr(step.kv_lens), _ptr(step.cu_seqlens), _ptr(out),
+                    step.num_seqs, work, H, G, D, page_size, float(scale), skip, chunk, _ptr(turns),
+                    _ptr(self._error_word(out.device)), self._stream())
+                if cost:
+                    cost(True)
+                    with self._timed("paged_attention_prefill_tc"):
+                        code = launch()
+                else:
+                    code = launch()
+                if code not in (0, 1):
+                    _check(code, "paged_attention_prefill_tc")
+                done = code == 0
+            if not done:
+                if cost:
+                    cost(True)
+                self._call("attention_chunk", "q3_chunk_attention_prefill", "chunk_attention_prefill", _ptr(q), q_stride,
+                           _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1], _ptr(step.kv_lens),
+                           _ptr(step.cu_seqlens), _ptr(out), out.stride(0), step.num_seqs,
+                           sum(-(-n * group // 128) for n in served), H, G, D, Dv, page_size, float(scale), chunk, skip,
+                           _ptr(turns), pairs, self.PAIRINGS[pairing])
+        if singles:
+            # the slice count comes from an upper bound of the lengths (in a captured step: the block-table width it
+            # was captured for), never from the lengths of the moment
+            bound = step.captured_width * page_size or step.max_kv_len
+            if chunk:
+                bound = min(bound, chunk + 63)
+            splits = max(1, min(-(-bound // 64), (3 * self.SM_COUNT) // max(1, singles * G), 64))
+            mid_o = mid_lse = tickets = None
+            if splits > 1 and singles * G > self.TICKETS:
+                splits = 1
+            if splits > 1:
+                padded = 64 if Dv <= 64 else (128 if Dv <= 128 else 256)
+                mid_o = torch.empty(singles * H * splits * padded, dtype=torch.float32, device=out.device)
+                mid_lse = torch.empty(singles * H * splits, dtype=torch.float32, device=out.device)
+                if self._tickets is None:  # zero between launches: the kernels leave them so
+                    self._tickets = torch.zeros(self.TICKETS, dtype=torch.int32, device=out.device)
+                tickets = self._tickets
+            if cost:
+                cost(False)
+            self._call("attention_chunk", "q3_chunk_attention_decode", "chunk_attention_decode", _ptr(q), q_stride,
+                       _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1], _ptr(step.kv_lens),
+                       _ptr(step.cu_seqlens), None if step.decode_only else _ptr(step.single_seqs), _ptr(out),
+                       out.stride(0), _ptr(mid_o), _ptr(mid_lse), _ptr(tickets), singles, H, G, D, Dv, page_size,
+                       float(scale), chunk, splits, _ptr(turns), pairs, self.PAIRINGS[pairing])
+        return out
+
+    @staticmethod
+    def _chunk_cost(step, H, G, D, Dv, chunk, out, prompts):
+        """(bytes, flops) of :meth:`_chunk_attention`: visible keys and values of each sequence read once, q read and the
+        result written; 2 * heads * (D + Dv) flops per visible (query, key) pair."""
+        e = out.element_size()
+        keys = pairs = rows = 0
+        cu = step.host_cu_seqlens
+        for b, kv in enumerate(step.host_kv_lens):
+            n = cu[b + 1] - cu[b] if len(cu) > b + 1 else 1
+            if (n > 1) != prompts:
+                continue
+            first = (kv - n) // chunk * chunk if chunk else 0
+            keys += kv - first
+            rows += n
+            if chunk:
+                pairs += sum(p % chunk + 1 for p in range(kv - n, kv))
+            else:
+                pairs += n * kv - n * (n - 1) // 2
+        return (keys * G * (D + Dv) + rows * H * (D + Dv)) * e, 2 * H * (D + Dv) * pairs
 
     def differential_attention(self, q, q_stride, *, num_heads, num_kv_heads, map_dim, value_dim, k_pages, v_pages,
                                block_table, token_seq, positions, out, page_size, scale, lam, eps, out_scale,

@@ -138,6 +138,10 @@ class SinkWindowAttention(BranchMixer):
     def kernel_groups(self):
         groups = ["rope_kv", "attention_generic"]
         groups += ["gemm_f32"] if self.ctx.dtype == torch.float32 else ["gemm_small_m", "gemm_stream"]
+        if self.turned and self.ctx.dtype == torch.bfloat16 and not self.window and self.sink is None and not self.gate:
+            groups.append("attention_chunk")
+            if self.dim == 128 and self.vdim == 128:
+                groups.append("attention_prefill_tc")
         if self._specialised():
             groups += ["attention_decode"] + (["attention_prefill"] if self.dim in (64, 128) else [])
         return groups
@@ -147,7 +151,7 @@ class SinkWindowAttention(BranchMixer):
         kernel (64, 128) take (ops.paged_attention sends a dense output there), with the window's kept first tokens, the
         sink, the gate and capped scores."""
         return (self.ctx.dtype == torch.bfloat16 and self.dim == self.vdim and self.dim in (64, 128, 256)
-                and self.num_heads // self.num_kv_heads <= 16 and not self.chunk)
+                and self.num_heads // self.num_kv_heads <= 16 and not self.chunk and self.value_position is None)
 
     # positions for which the decode kernel that also makes the newest token's q and k keeps rotation tables;
     # steps that reach beyond run the q/k kernel (which needs none) and the plain decode kernel

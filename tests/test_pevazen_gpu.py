@@ -169,3 +169,34 @@ def test_command_line_on_a_pevazen_folder(tmp_path):
         row = pl.forward(raw, t, seq)[-1].float()
         assert float(row.max() - row[tok]) <= 1e-4 * max(1.0, float(row.abs().max()))
         seq.append(tok)
+
+
+def test_bfloat16_steps_take_the_specialised_kernels(tmp_path, ops):
+    """A bfloat16 model runs prompt portions on the tensor-core kernels (tcgen05 for heads of 128) and decode steps on
+    the kernel over slices of the visible keys and the kernel that does a whole delta-rule step; the general attention
+    kernel is not launched."""
+    from helpers import run_trace, trace_tail_decode
+
+    folder = pc.make_dir(tmp_path, "D")
+    launched = []
+    call, timed, ops.timing = ops._call, ops._timed, []
+
+    def call_spy(group, name, what, *args):
+        launched.append(what)
+        return call(group, name, what, *args)
+
+    def timed_spy(what):  # launches that may be refused go past _call
+        launched.append(what)
+        return timed(what)
+
+    ops._call, ops._timed = call_spy, timed_spy
+    try:
+        rt = pc.runtime(folder, "D", "bfloat16", ops, DEV, pages=16)
+        run_trace(rt, trace_tail_decode(pc.requests_for("D", (70,)), tail=5))
+    finally:
+        del ops._call, ops._timed
+        ops.timing = None
+    for kernel in ("paged_attention_prefill_tc", "chunk_attention_prefill", "chunk_attention_decode", "delta_step",
+                   "delta_prepare", "turn_store", "sum_norm", "embed_norm"):
+        assert kernel in launched, f"{kernel} was not launched: {sorted(set(launched))}"
+    assert "paged_attention" not in launched
