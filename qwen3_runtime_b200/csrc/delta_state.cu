@@ -14,6 +14,7 @@
 //   delta_prepare    every token of a step: convolution, silu, unit vectors, decays and steps as rows in memory
 //   ring_update      the last rows of every sequence's portion into the ring (after delta_prepare has read it)
 //   delta_scan       the recurrence over every sequence's tokens of the step, from delta_prepare's rows
+//   delta_chunk_*    the same in chunks of 16 tokens, for prompts
 //   delta_step       all of it for steps in which every sequence brings one token, with the decay's and the
 //                    gate's second low-rank products and the heads' output norm and gate: one kernel
 #include "common.cuh"
@@ -367,6 +368,325 @@ Q3_EXPORT int q3_delta_scan(int dtype, const float* qn, const float* kn, const v
 #undef Q3_DELTA_SIZES
 #undef Q3_DELTA_SCAN
   return e == cudaSuccess ? Q3_OK : Q3_ERR_LAUNCH;
+}
+
+// ---- the recurrence in chunks of 16 tokens ------------------------------------------------------------
+// With G_i the product of a chunk's decays up to token i and S the state before the chunk, the recurrence is, in
+// matrices whose rows are the chunk's tokens (the WY form of a product of rank-one updates):
+//   A_ij = sum_d k_i k_j prod_(j < m <= i) g_m  (j < i)        B_ij = sum_d q_i k_j prod_(j < m <= i) g_m  (j <= i)
+//   W = (I + diag(beta) A)^(-1) diag(beta)
+//   U = W (V - (G k) S)      O = (G q) S + B U      S <- G_last S + sum_j (prod_(m > j) g_m k_j) u_j^T
+// Only products of decays occur, never quotients, so strong decays lose nothing.  All of it is fp32 FMA.
+//
+// delta_chunk_rows: everything that does not depend on the state, a record of DC_REC floats per (chunk, head):
+// [DP][32] (G k | G q, transposed), [16][DP] the decayed-to-the-end keys, [DP] G_last, W and B [16][16].  Chunks of
+// sequence b start at place cu_seqlens[b] / 16 + b; tokens beyond a portion's end are k = q = 0, g = 1, beta = 0.
+// delta_chunk_scan: one block per (16 value columns, head, sequence); the state's columns stay in registers (and, for
+// the products with it, in shared memory), the next chunk's record is on its way while one is worked on.
+#define DC_C 16
+#define DC_REC(DP) ((DP) * 49 + 2 * DC_C * DC_C)
+
+template <int DP>
+__global__ void __launch_bounds__(256)
+delta_chunk_rows_kernel(const float* __restrict__ qn, const float* __restrict__ kn, const float* __restrict__ g,
+                        const float* __restrict__ beta, const int* __restrict__ cu_seqlens, int num_seqs,
+                        float* __restrict__ records, int G, int H, int D) {
+  __shared__ __align__(16) float ks[DC_C][DP], qs[DC_C][DP], gs[DC_C][DP];
+  __shared__ float as[DC_C][DC_C + 1], bs[DC_C][DC_C + 1], be[DC_C];
+  __shared__ int s_t0, s_n;
+  pdl_wait();
+  pdl_launch_dependents();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int place = blockIdx.x, h = blockIdx.y, gh = h / (H / G);
+  if (tid == 0) {
+    int n = 0, t0 = 0;
+    for (int b = 0; b < num_seqs; ++b) {
+      const int c0 = cu_seqlens[b], c1 = cu_seqlens[b + 1], base = c0 / DC_C + b;
+      if (place >= base && place < c1 / DC_C + b + 1) {
+        t0 = c0 + (place - base) * DC_C;
+        n = c1 - t0;
+        break;
+      }
+    }
+    s_t0 = t0;
+    s_n = n > DC_C ? DC_C : n;
+  }
+  __syncthreads();
+  const int n = s_n;
+  const long t0 = s_t0;
+  if (n <= 0) return;
+  for (int x = tid; x < DC_C * DP; x += 256) {
+    const int c = x / DP, i = x - c * DP;
+    const bool live = c < n && i < D;
+    ks[c][i] = live ? kn[((t0 + c) * G + gh) * D + i] : 0.f;
+    qs[c][i] = live ? qn[((t0 + c) * G + gh) * D + i] : 0.f;
+    gs[c][i] = live ? g[((t0 + c) * H + h) * D + i] : 1.f;
+  }
+  if (tid < DC_C) be[tid] = tid < n ? beta[(t0 + tid) * H + h] : 0.f;
+  __syncthreads();
+  float* rec = records + ((long)place * H + h) * DC_REC(DP);
+  if (tid < DP) {  // the keys and queries decayed from the chunk's start, a channel's 32 values side by side
+    float* dst = rec + tid * 32;
+    float run = 1.f;
+#pragma unroll
+    for (int c = 0; c < DC_C; c += 4) {
+      float a[4], b[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        run *= gs[c + e][tid];
+        a[e] = run * ks[c + e][tid];
+        b[e] = run * qs[c + e][tid];
+      }
+      *reinterpret_cast<float4*>(dst + c) = make_float4(a[0], a[1], a[2], a[3]);
+      *reinterpret_cast<float4*>(dst + DC_C + c) = make_float4(b[0], b[1], b[2], b[3]);
+    }
+    rec[48 * DP + tid] = run;
+  } else if (tid < 2 * DP) {  // the keys decayed to the chunk's end
+    const int i = tid - DP;
+    float run = 1.f;
+#pragma unroll
+    for (int c = DC_C - 1; c >= 0; --c) {
+      rec[32 * DP + c * DP + i] = run * ks[c][i];
+      run *= gs[c][i];
+    }
+  }
+  constexpr int E = DP / 32;
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {  // rows i and 15 - i: every warp the same work
+    const int i = half ? DC_C - 1 - warp : warp;
+    float wk[E], wq[E];
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+      wk[e] = ks[i][lane + 32 * e];
+      wq[e] = qs[i][lane + 32 * e];
+    }
+    for (int j = i; j >= 0; --j) {
+      float a = 0.f, b = 0.f;
+#pragma unroll
+      for (int e = 0; e < E; ++e) {
+        const float kj = ks[j][lane + 32 * e];
+        a = fmaf(wk[e], kj, a);
+        b = fmaf(wq[e], kj, b);
+        const float gj = gs[j][lane + 32 * e];
+        wk[e] *= gj;
+        wq[e] *= gj;
+      }
+      a = warp_sum(a);
+      b = warp_sum(b);
+      if (lane == 0) {
+        as[i][j] = a;  // (the diagonal is not used)
+        bs[i][j] = b;
+      }
+    }
+  }
+  __syncthreads();
+  if (tid < DC_C) {  // column tid of W by forward substitution
+    float x[DC_C];
+#pragma unroll
+    for (int i = 0; i < DC_C; ++i) {
+      float acc = i == tid ? 1.f : 0.f;
+#pragma unroll
+      for (int j = 0; j < i; ++j) acc = fmaf(-as[i][j], x[j], acc);
+      x[i] = be[i] * acc;
+      rec[49 * DP + i * DC_C + tid] = x[i];
+    }
+  } else if (tid >= 64 && tid < 64 + DC_C * 4) {
+    const int i = (tid - 64) >> 2, j0 = ((tid - 64) & 3) * 4;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) rec[49 * DP + DC_C * DC_C + i * DC_C + j0 + e] = j0 + e <= i ? bs[i][j0 + e] : 0.f;
+  }
+}
+
+__device__ __forceinline__ void ds_copy16(float* dst, const float* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src));
+}
+
+template <typename T, int DP>
+__global__ void __launch_bounds__(256)
+delta_chunk_scan_kernel(const float* __restrict__ records, const T* __restrict__ vc, float* __restrict__ state,
+                        const int* __restrict__ cu_seqlens, const int* __restrict__ state_slots, float* __restrict__ out,
+                        int H, int D, int Dv) {
+  constexpr int VT = 16, REC = DC_REC(DP), RD = DP / 64, PS = 20;  // PS: row pitch of the partial sums
+  extern __shared__ __align__(16) float dc_smem[];
+  float* Ss = dc_smem + 2 * REC;       // [DP][VT]
+  float* part = Ss + DP * VT;          // [8][32][PS]
+  float* ys = part + 8 * 32 * PS;      // [16][VT]
+  float* us = ys + DC_C * VT;          // [16][VT]
+  pdl_wait();
+  pdl_launch_dependents();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int h = blockIdx.y, b = blockIdx.z, col0 = blockIdx.x * VT;
+  const int t0 = cu_seqlens[b], t1 = cu_seqlens[b + 1];
+  if (t1 <= t0) return;
+  const int chunks = (t1 - t0 + DC_C - 1) / DC_C;
+  const float* rec0 = records + ((long)(t0 / DC_C + b) * H + h) * REC;
+  auto load = [&](int c) {
+    const float* src = rec0 + (long)c * H * REC;
+    float* dst = dc_smem + (c & 1) * REC;
+    for (int x = tid * 4; x < REC; x += 1024) ds_copy16(dst + x, src + x);
+    asm volatile("cp.async.commit_group;\n" ::);
+  };
+  load(0);
+  // this thread's rows and columns of the state
+  const int d0 = (tid >> 2) * RD, c0 = (tid & 3) * 4;
+  float* Sg = state + ((long)state_slots[b] * H + h) * (long)D * Dv;
+  float S[RD][4];
+#pragma unroll
+  for (int r = 0; r < RD; ++r) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      S[r][e] = d0 + r < D && col0 + c0 + e < Dv ? Sg[(long)(d0 + r) * Dv + col0 + c0 + e] : 0.f;
+    *reinterpret_cast<float4*>(Ss + (d0 + r) * VT + c0) = make_float4(S[r][0], S[r][1], S[r][2], S[r][3]);
+  }
+  const int row = tid >> 4, col = tid & 15;  // the chunk's token and the value column of the small products
+  const bool col_in = col0 + col < Dv;
+  auto value = [&](int c) {
+    const long t = t0 + c * DC_C + row;
+    return col_in && t < t1 ? to_f32(vc[(t * H + h) * Dv + col0 + col]) : 0.f;
+  };
+  float v_next = value(0);
+  const int rt = (lane >> 2) * 4, ct = (lane & 3) * 4;
+  for (int c = 0; c < chunks; ++c) {
+    asm volatile("cp.async.wait_group 0;\n" ::);
+    __syncthreads();  // the record and the state in shared memory are complete; nobody reads the other record
+    const float* rec = dc_smem + (c & 1) * REC;
+    const float v = v_next;
+    if (c + 1 < chunks) {
+      load(c + 1);
+      v_next = value(c + 1);
+    }
+    {  // [G k; G q] S, an eighth of the channels a warp, 4 x 4 sums a thread
+      float acc[4][4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+#pragma unroll
+      for (int dd = 0; dd < DP / 8; ++dd) {
+        const int d = warp * (DP / 8) + dd;
+        const float4 a = *reinterpret_cast<const float4*>(rec + d * 32 + rt);
+        const float4 s = *reinterpret_cast<const float4*>(Ss + d * VT + ct);
+        const float av[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          acc[i][0] = fmaf(av[i], s.x, acc[i][0]);
+          acc[i][1] = fmaf(av[i], s.y, acc[i][1]);
+          acc[i][2] = fmaf(av[i], s.z, acc[i][2]);
+          acc[i][3] = fmaf(av[i], s.w, acc[i][3]);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        *reinterpret_cast<float4*>(part + (warp * 32 + rt + i) * PS + ct) =
+            make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+    }
+    __syncthreads();
+    float pk = 0.f, o = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) {
+      pk += part[(w * 32 + row) * PS + col];
+      o += part[(w * 32 + 16 + row) * PS + col];
+    }
+    ys[row * VT + col] = v - pk;
+    __syncthreads();
+    {
+      const float* W = rec + 49 * DP + row * DC_C;
+      float u = 0.f;
+#pragma unroll
+      for (int j = 0; j < DC_C; j += 4) {  // (W is zero beyond the diagonal)
+        const float4 w4 = *reinterpret_cast<const float4*>(W + j);
+        u = fmaf(w4.x, ys[j * VT + col], u);
+        u = fmaf(w4.y, ys[(j + 1) * VT + col], u);
+        u = fmaf(w4.z, ys[(j + 2) * VT + col], u);
+        u = fmaf(w4.w, ys[(j + 3) * VT + col], u);
+      }
+      us[row * VT + col] = u;
+    }
+    __syncthreads();
+    {
+      const float* B = rec + 49 * DP + DC_C * DC_C + row * DC_C;
+#pragma unroll
+      for (int j = 0; j < DC_C; j += 4) {
+        const float4 b4 = *reinterpret_cast<const float4*>(B + j);
+        o = fmaf(b4.x, us[j * VT + col], o);
+        o = fmaf(b4.y, us[(j + 1) * VT + col], o);
+        o = fmaf(b4.z, us[(j + 2) * VT + col], o);
+        o = fmaf(b4.w, us[(j + 3) * VT + col], o);
+      }
+      const long t = t0 + c * DC_C + row;
+      if (col_in && t < t1) out[(t * H + h) * Dv + col0 + col] = o;
+    }
+    const float* kend = rec + 32 * DP;
+#pragma unroll
+    for (int r = 0; r < RD; ++r) {
+      const float gl = rec[48 * DP + d0 + r];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) S[r][e] *= gl;
+    }
+#pragma unroll
+    for (int j = 0; j < DC_C; ++j) {
+      const float4 u4 = *reinterpret_cast<const float4*>(us + j * VT + c0);
+#pragma unroll
+      for (int r = 0; r < RD; ++r) {
+        const float kk = kend[j * DP + d0 + r];
+        S[r][0] = fmaf(kk, u4.x, S[r][0]);
+        S[r][1] = fmaf(kk, u4.y, S[r][1]);
+        S[r][2] = fmaf(kk, u4.z, S[r][2]);
+        S[r][3] = fmaf(kk, u4.w, S[r][3]);
+      }
+    }
+#pragma unroll
+    for (int r = 0; r < RD; ++r)
+      *reinterpret_cast<float4*>(Ss + (d0 + r) * VT + c0) = make_float4(S[r][0], S[r][1], S[r][2], S[r][3]);
+  }
+#pragma unroll
+  for (int r = 0; r < RD; ++r)
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      if (d0 + r < D && col0 + c0 + e < Dv) Sg[(long)(d0 + r) * Dv + col0 + c0 + e] = S[r][e];
+}
+
+template <typename T, int DP>
+static int launch_delta_chunks(cudaStream_t stream, int num_tokens, int num_seqs, const float* qn, const float* kn,
+                               const void* vc, const float* g, const float* beta, float* records, float* state,
+                               const int* cu_seqlens, const int* state_slots, float* out, int G, int H, int D, int Dv) {
+  const int places = num_tokens / DC_C + num_seqs;
+  if (launch_pdl(delta_chunk_rows_kernel<DP>, dim3(places, H), dim3(256), 0, stream, qn, kn, g, beta, cu_seqlens, num_seqs,
+                 records, G, H, D) != cudaSuccess)
+    return Q3_ERR_LAUNCH;
+  constexpr size_t smem = sizeof(float) * (2 * DC_REC(DP) + DP * 16 + 8 * 32 * 20 + 2 * DC_C * 16);
+  auto kernel = delta_chunk_scan_kernel<T, DP>;
+  static bool configured_on[Q3_MAX_DEVICES];
+  bool& configured = configured_on[q3_current_device()];
+  if (!configured) {
+    if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+      return Q3_ERR_LAUNCH;
+    configured = true;
+  }
+  return launch_pdl(kernel, dim3((Dv + 15) / 16, H, num_seqs), dim3(256), smem, stream, (const float*)records, (const T*)vc,
+                    state, cu_seqlens, state_slots, out, H, D, Dv) == cudaSuccess
+             ? Q3_OK
+             : Q3_ERR_LAUNCH;
+}
+
+// The same as q3_delta_scan for key sizes up to 128, in chunks; records: (num_tokens / 16 + num_seqs) * H * (49 * DP +
+// 512) floats with DP = 64 (D <= 64) or 128.
+Q3_EXPORT int q3_delta_chunk_scan(int dtype, const float* qn, const float* kn, const void* vc, const float* g,
+                                  const float* beta, float* records, float* state, const int* cu_seqlens,
+                                  const int* state_slots, float* out, int num_tokens, int num_seqs, int G, int H, int D,
+                                  int Dv, cudaStream_t stream) {
+  if (!qn || !kn || !vc || !g || !beta || !records || !state || !cu_seqlens || !state_slots || !out) return Q3_ERR_ARGUMENT;
+  if (G < 1 || H < 1 || H % G || D < 1 || Dv < 1 || H > 65535 || num_seqs > 65535) return Q3_ERR_ARGUMENT;
+  if (D > 128 || (dtype != Q3_DTYPE_F32 && dtype != Q3_DTYPE_BF16) || !ds_aligned(records)) return Q3_ERR_UNSUPPORTED;
+  if (num_seqs == 0 || num_tokens == 0) return Q3_OK;
+#define Q3_DELTA_CHUNKS(T, DP)                                                                                       \
+  return launch_delta_chunks<T, DP>(stream, num_tokens, num_seqs, qn, kn, vc, g, beta, records, state, cu_seqlens,   \
+                                    state_slots, out, G, H, D, Dv)
+  if (dtype == Q3_DTYPE_F32) {
+    if (D <= 64) Q3_DELTA_CHUNKS(float, 64);
+    Q3_DELTA_CHUNKS(float, 128);
+  }
+  if (D <= 64) Q3_DELTA_CHUNKS(bf16, 64);
+  Q3_DELTA_CHUNKS(bf16, 128);
+#undef Q3_DELTA_CHUNKS
 }
 
 // ---- steps in which every sequence brings one token, in one kernel ------------------------------------

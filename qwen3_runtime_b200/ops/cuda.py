@@ -137,6 +137,8 @@ _SIGNATURES = {
                            c_void_p],
         "q3_delta_scan": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                           c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
+        "q3_delta_chunk_scan": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p],
         "q3_delta_step": [c_int, c_void_p, c_long, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                           c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p,
                           c_void_p, c_float, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_void_p],
@@ -284,6 +286,7 @@ class CudaOps:
         self.latent_attention_tc = True     # False: attention over latent rows always on the general kernel
         self.experts_tc = True              # False: the experts' products always on the FMA kernels
         self.chunk_tc = True                # False: attention under chunks or with turned values on the general kernel
+        self.delta_chunks = True            # False: the delta rule's recurrence always token by token
         self.differential_tc = True         # False: differential attention always on the general kernel
         self._tickets: torch.Tensor | None = None
         self._argmax_tickets: torch.Tensor | None = None
@@ -830,6 +833,15 @@ class CudaOps:
         if self.timing is not None:
             self._costs(2 * num_seqs * H * D * Dv * 4 + T * (8 * G * D + H * Dv * (e + 4) + 4 * H * D),
                         7.0 * T * H * D * Dv)
+        if self.delta_chunks and D <= 128 and T >= max(32, 4 * num_seqs):
+            # prompts: chunks of 16 tokens (csrc/delta_state.cu); what does not depend on the state first
+            padded = 64 if D <= 64 else 128
+            records = torch.empty((T // 16 + num_seqs) * H * (49 * padded + 512), dtype=torch.float32, device=dev)
+            self.launches += 1
+            self._call("delta_state", "q3_delta_chunk_scan", "delta_chunk_scan", _dtype_code(x.dtype), _ptr(qn), _ptr(kn),
+                       _ptr(vc), _ptr(g), _ptr(beta), _ptr(records), _ptr(state), _ptr(cu_seqlens), _ptr(state_slots),
+                       _ptr(out), T, int(num_seqs), G, H, D, Dv)
+            return out
         self._call("delta_state", "q3_delta_scan", "delta_scan", _dtype_code(x.dtype), _ptr(qn), _ptr(kn), _ptr(vc),
                    _ptr(g), _ptr(beta), _ptr(state), _ptr(cu_seqlens), _ptr(state_slots), _ptr(out), int(num_seqs), G, H,
                    D, Dv)

@@ -69,6 +69,15 @@ def test_delta_rule(ops, dtype):
     pc.case_delta_rule(dtype, ops, DEV, H=2, G=2, D=64, Dv=64, taps=2, ra=16, rg=8)
     pc.case_delta_rule(dtype, ops, DEV, H=4, G=1, D=128, Dv=128, taps=4, ra=32, rg=16, lens=(130, 3, 33, 16))
     pc.case_delta_rule(dtype, ops, DEV, H=2, G=1, D=128, Dv=40, taps=3, ra=8, rg=8, lens=(300, 17, 1), decay=-5.0)
+    # chunks of 16 tokens: portions on both sides of a chunk's edge, very strong and very weak decays, many sequences
+    pc.case_delta_rule(dtype, ops, DEV, H=3, G=1, D=72, Dv=24, taps=4, ra=8, rg=8, lens=(15, 16, 17, 33, 64), decay=4.0)
+    pc.case_delta_rule(dtype, ops, DEV, H=2, G=1, D=40, Dv=100, taps=2, ra=8, rg=8, lens=(31, 1, 48, 2, 1, 65), decay=-6.0)
+    ops.delta_chunks = False  # the same sizes token by token
+    try:
+        pc.case_delta_rule(dtype, ops, DEV, H=4, G=1, D=128, Dv=128, taps=4, ra=32, rg=16, lens=(130, 3, 33, 16))
+        pc.case_delta_rule(dtype, ops, DEV, H=3, G=1, D=72, Dv=24, taps=4, ra=8, rg=8, lens=(15, 16, 17, 33, 64), decay=4.0)
+    finally:
+        ops.delta_chunks = True
     pc.case_delta_rule(dtype, ops, DEV, H=2, G=2, D=200, Dv=136, taps=5, ra=8, rg=8, lens=(40, 1, 5))
     pc.case_delta_rule(dtype, ops, DEV, H=2, G=2, D=32, Dv=256, taps=4, ra=8, rg=12, lens=(40, 1, 5), decay=3.0)
 
@@ -197,6 +206,6 @@ def test_bfloat16_steps_take_the_specialised_kernels(tmp_path, ops):
         del ops._call, ops._timed
         ops.timing = None
     for kernel in ("paged_attention_prefill_tc", "chunk_attention_prefill", "chunk_attention_decode", "delta_step",
-                   "delta_prepare", "turn_store", "sum_norm", "embed_norm"):
+                   "delta_prepare", "delta_chunk_scan", "turn_store", "sum_norm", "embed_norm"):
         assert kernel in launched, f"{kernel} was not launched: {sorted(set(launched))}"
     assert "paged_attention" not in launched
