@@ -22,8 +22,7 @@ constexpr int TILE = 64;
 
 __device__ __forceinline__ int first_seen(int p, int chunk) { return chunk > 0 ? p / chunk * chunk : 0; }
 
-// One row of `dv` fp32 values in shared memory, turned back by cs = [cos(pairs) | sin(pairs)] (null: as they are), two
-// neighbouring elements a call.
+// Element d of a row of fp32 values in shared memory, turned back by cs = [cos(pairs) | sin(pairs)] (null: as it is).
 __device__ __forceinline__ float turned_back(const float* row, int d, const float* cs, int pairs, int pairing) {
   const float v = row[d];
   if (!cs || d >= 2 * pairs) return v;
