@@ -4,6 +4,7 @@ from .medilix_config import MedilixConfig
 from .puladra_config import PuladraConfig
 from .tabisun_config import TabisunConfig
 from .pevazen_config import PevazenConfig
+from .timopel_config import TimopelConfig
 from .model_config import ConfigError, Qwen3Config
 from .registry import (
     Architecture,
@@ -33,6 +34,7 @@ __all__ = [
     "PuladraConfig",
     "Qwen3Config",
     "TabisunConfig",
+    "TimopelConfig",
     "canonical_dtype",
     "load_config",
     "read_config_json",

@@ -1,7 +1,8 @@
 // Attention over the paged cache in bfloat16 for keys and values of sizes of their own, under a chunked mask, with
 // values that may be turned by their positions.  A token at position p sees keys lo .. p with lo = floor(p / chunk) *
 // chunk (chunk > 0; chunks counted from the sequence's first token) or 0.  With turn tables the cached values are
-// turned by their own positions, and a head's sum is turned back by the token's angles before it is stored.
+// turned by their own positions, and a head's sum is turned back by the token's angles before it is stored.  With
+// sinks (fp32, one score per head) each softmax's denominator has one more term, exp(sink_h), that stands for no key.
 // Key pages [pages, nkv, ps, D], value pages [pages, nkv, ps, DV]; D and DV multiples of 8 up to 256.  The kernels
 // are made for DP, DVP in {64, 128, 256}; columns between a size and its DP are zeros in shared memory.
 //
@@ -44,7 +45,8 @@ chunk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __res
                      const bf16* __restrict__ vpages, const int* __restrict__ block_table, int max_pages,
                      const int* __restrict__ kv_lens, const int* __restrict__ cu_seqlens, bf16* __restrict__ out,
                      long out_stride, int num_seqs, int nq, int nkv, int D, int DV, int ps, float scale_log2, int chunk,
-                     int skip_single, const float* __restrict__ turns, int pairs, int pairing) {
+                     int skip_single, const float* __restrict__ turns, int pairs, int pairing,
+                     const float* __restrict__ sinks) {
   constexpr int STAGES = prefill_stages<DP, DVP>();
   constexpr int KCH = DP / 8, VCH = DVP / 8;
   constexpr int K_BYTES = TILE * DP * 2, V_BYTES = TILE * DVP * 2;
@@ -244,6 +246,8 @@ chunk_prefill_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __res
   for (int r = 0; r < 2; ++r) {
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
+    const int R = row0 + warp * 16 + (lane >> 2) + r * 8;
+    if (sinks && R < rows) l_run[r] += exp2f(sinks[kvh * G + R % G] * LOG2_E - m_run[r] * scale_log2);
     inv[r] = l_run[r] > 0.f ? 1.f / l_run[r] : 0.f;
   }
   if (!turns) {
@@ -286,7 +290,8 @@ template <int DP, int DVP>
 int launch_chunk_prefill(const bf16* q, int q_stride, const bf16* kpages, const bf16* vpages, const int* block_table,
                          int max_pages, const int* kv_lens, const int* cu_seqlens, bf16* out, long out_stride,
                          int num_seqs, int num_work, int nq, int nkv, int D, int DV, int ps, float scale, int chunk,
-                         int skip_single, const float* turns, int pairs, int pairing, cudaStream_t stream) {
+                         int skip_single, const float* turns, int pairs, int pairing, const float* sinks,
+                         cudaStream_t stream) {
   const size_t pipe = (size_t)BLOCK_M * DP * 2 + (size_t)prefill_stages<DP, DVP>() * TILE * (DP + DVP) * 2;
   const size_t rows = (size_t)BLOCK_M * (DVP + 8) * 4;
   const size_t smem = pipe > rows ? pipe : rows;
@@ -300,7 +305,7 @@ int launch_chunk_prefill(const bf16* q, int q_stride, const bf16* kpages, const 
   }
   chunk_prefill_kernel<DP, DVP><<<dim3(num_work, nkv), PF_THREADS, smem, stream>>>(
       q, q_stride, kpages, vpages, block_table, max_pages, kv_lens, cu_seqlens, out, out_stride, num_seqs, nq, nkv, D, DV,
-      ps, scale * 1.4426950408889634f, chunk, skip_single, turns, pairs, pairing);
+      ps, scale * 1.4426950408889634f, chunk, skip_single, turns, pairs, pairing, sinks);
   return q3_launch_status();
 }
 
@@ -318,7 +323,7 @@ chunk_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
                     const int* __restrict__ kv_lens, const int* __restrict__ cu_seqlens, const int* __restrict__ seq_list,
                     bf16* __restrict__ out, long out_stride, float* mid_o, float* mid_lse, int* tickets, int nq, int nkv,
                     int D, int DV, int ps, float scale_log2, int chunk, int splits, const float* __restrict__ turns,
-                    int pairs, int pairing) {
+                    int pairs, int pairing, const float* __restrict__ sinks) {
   constexpr int KCH = DP / 8, VCH = DVP / 8;
   constexpr int K_BYTES = TILE * DP * 2, V_BYTES = TILE * DVP * 2;
   extern __shared__ __align__(128) unsigned char smem[];
@@ -500,10 +505,11 @@ chunk_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
       l += ml_s[(w * 16 + g) * 2 + 1] * f;
       acc += o_s[((size_t)w * 16 + g) * OS + d] * f;
     }
-    const float val = l > 0.f ? acc / l : 0.f;
     if (slices == 1) {
-      fin[g * DVP + d] = val;
+      if (sinks) l += exp2f(sinks[kvh * G + g] * LOG2_E - m * scale_log2);
+      fin[g * DVP + d] = acc / l;
     } else {
+      const float val = l > 0.f ? acc / l : 0.f;
       mid_o[((item * G + g) * splits + split) * DVP + d] = val;
       if (d == 0) mid_lse[(item * G + g) * splits + split] = l > 0.f ? m * scale_log2 + log2f(l) : -INFINITY;
     }
@@ -524,7 +530,7 @@ chunk_decode_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __rest
       const float* src = mid_o + (item * G + g) * splits * DVP + d;
       float mx = -INFINITY;
       for (int s = 0; s < slices; ++s) mx = fmaxf(mx, __ldcg(lse + s));
-      float acc = 0.f, wsum = 0.f;
+      float acc = 0.f, wsum = sinks ? exp2f(sinks[kvh * G + g] * LOG2_E - mx) : 0.f;
 #pragma unroll 4
       for (int s = 0; s < slices; ++s) {
         const float w = exp2f(__ldcg(lse + s) - mx);
@@ -549,7 +555,7 @@ int launch_chunk_decode(const bf16* q, int q_stride, const bf16* kpages, const b
                         int max_pages, const int* kv_lens, const int* cu_seqlens, const int* seq_list, bf16* out,
                         long out_stride, float* mid_o, float* mid_lse, int* tickets, int num_seqs, int nq, int nkv, int D,
                         int DV, int ps, float scale, int chunk, int splits, const float* turns, int pairs, int pairing,
-                        cudaStream_t stream) {
+                        const float* sinks, cudaStream_t stream) {
   const size_t pipe = (size_t)2 * TILE * (DP + DVP) * 2;
   const size_t merge = ((size_t)DC_WARPS * 16 * (DVP + 8) + DC_WARPS * 32 + 16 * DVP) * 4;
   const size_t smem = 16 * DP * 2 + (pipe > merge ? pipe : merge);
@@ -564,7 +570,7 @@ int launch_chunk_decode(const bf16* q, int q_stride, const bf16* kpages, const b
   return launch_pdl(chunk_decode_kernel<DP, DVP>, dim3(splits, nkv, num_seqs), dim3(DC_THREADS), smem, stream, q, q_stride,
                     kpages, vpages, block_table, max_pages, kv_lens, cu_seqlens, seq_list, out, out_stride, mid_o, mid_lse,
                     tickets, nq, nkv, D, DV, ps, scale * 1.4426950408889634f, chunk, splits, turns, pairs,
-                    pairing) == cudaSuccess
+                    pairing, sinks) == cudaSuccess
              ? Q3_OK
              : Q3_ERR_LAUNCH;
 }
@@ -586,12 +592,14 @@ bool chunk_sizes_ok(const void* q, int q_stride, const void* kpages, const void*
   CALL(256, 256);
 
 // Prompt portions: num_work = sum over the served sequences of ceil(q_len * (nq / nkv) / 128); with skip_single the
-// sequences of one token are left out.  turns: null, or fp32 [num_tokens, 2, pairs].  Groups of at most 16 heads.
+// sequences of one token are left out.  turns: null, or fp32 [num_tokens, 2, pairs].  sinks: null, or fp32
+// [nq].  Groups of at most 16 heads.
 Q3_EXPORT int q3_chunk_attention_prefill(const void* q, int q_stride, const void* kpages, const void* vpages,
                                          const int* block_table, int max_pages, const int* kv_lens,
                                          const int* cu_seqlens, void* out, long out_stride, int num_seqs, int num_work,
                                          int nq, int nkv, int D, int DV, int ps, float scale, int chunk, int skip_single,
-                                         const float* turns, int pairs, int pairing, cudaStream_t stream) {
+                                         const float* turns, int pairs, int pairing, const float* sinks,
+                                         cudaStream_t stream) {
   if (!q || !kpages || !vpages || !block_table || !kv_lens || !cu_seqlens || !out) return Q3_ERR_ARGUMENT;
   if (nq < 1 || nkv < 1 || nq % nkv || ps < 1 || num_seqs < 0 || num_work < 0 || chunk < 0) return Q3_ERR_ARGUMENT;
   if (turns && (pairs < 1 || 2 * pairs > DV || pairing < 0 || pairing > 1)) return Q3_ERR_ARGUMENT;
@@ -600,7 +608,7 @@ Q3_EXPORT int q3_chunk_attention_prefill(const void* q, int q_stride, const void
 #define Q3_CHUNK_PREFILL(dp, dvp)                                                                                     \
   return launch_chunk_prefill<dp, dvp>((const bf16*)q, q_stride, (const bf16*)kpages, (const bf16*)vpages, block_table, \
                                        max_pages, kv_lens, cu_seqlens, (bf16*)out, out_stride, num_seqs, num_work, nq, nkv, \
-                                       D, DV, ps, scale, chunk, skip_single, turns, pairs, pairing, stream)
+                                       D, DV, ps, scale, chunk, skip_single, turns, pairs, pairing, sinks, stream)
   Q3_CHUNK_SIZES(Q3_CHUNK_PREFILL)
 #undef Q3_CHUNK_PREFILL
 }
@@ -613,7 +621,7 @@ Q3_EXPORT int q3_chunk_attention_decode(const void* q, int q_stride, const void*
                                         const int* seq_list, void* out, long out_stride, float* mid_o, float* mid_lse,
                                         int* tickets, int num_seqs, int nq, int nkv, int D, int DV, int ps, float scale,
                                         int chunk, int splits, const float* turns, int pairs, int pairing,
-                                        cudaStream_t stream) {
+                                        const float* sinks, cudaStream_t stream) {
   if (!q || !kpages || !vpages || !block_table || !kv_lens || !cu_seqlens || !out) return Q3_ERR_ARGUMENT;
   if (nq < 1 || nkv < 1 || nq % nkv || ps < 1 || num_seqs < 0 || splits < 1 || chunk < 0) return Q3_ERR_ARGUMENT;
   if (splits > 1 && (!mid_o || !mid_lse || !tickets)) return Q3_ERR_ARGUMENT;
@@ -625,7 +633,7 @@ Q3_EXPORT int q3_chunk_attention_decode(const void* q, int q_stride, const void*
   return launch_chunk_decode<dp, dvp>((const bf16*)q, q_stride, (const bf16*)kpages, (const bf16*)vpages, block_table, \
                                       max_pages, kv_lens, cu_seqlens, seq_list, (bf16*)out, out_stride, mid_o, mid_lse, \
                                       tickets, num_seqs, nq, nkv, D, DV, ps, scale, chunk, splits, turns, pairs, pairing, \
-                                      stream)
+                                      sinks, stream)
   Q3_CHUNK_SIZES(Q3_CHUNK_DECODE)
 #undef Q3_CHUNK_DECODE
 }

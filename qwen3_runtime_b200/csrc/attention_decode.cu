@@ -43,20 +43,27 @@ struct NewToken {
   int max_pos;
   int pairing;
   int v_from_k;
+  const float* q_scale;  // null, or a factor per packed token for its queries (after norm and rotation)
+  const bf16* v_first;   // null, or rows of nkv value heads per packed token, v_first_stride apart, of which the newest
+  int v_first_stride;    // token's value takes the share v_share: v <- (1 - v_share) v + v_share v_first
+  float v_share;
 };
 
 // What some designs add to the attention.  keep: with a window, the sequence's first `keep` tokens stay
-// visible.  sink_log2: a score (times log2 e) that has no value and joins the softmax's denominator; minus
-// infinity for none.  gate: null, or rows [tokens][gate_stride] whose first heads * D values gate the result
+// visible.  sinks: null, or per head (fp32 [nq]) a score that has no value and joins the softmax's denominator.
+// gate: null, or rows [tokens][gate_stride] whose first heads * D values gate the result
 // by their sigmoid.  cap_raw: scores are capped, score <- cap * tanh(score / cap) after the scale; given in the
 // unscaled dot product's units (cap / scale), 0 for none.
 struct Extras {
   int keep = 0;
-  float sink_log2 = -INFINITY;
+  const float* sinks = nullptr;
   const bf16* gate = nullptr;
   int gate_stride = 0;
   float cap_raw = 0.f;
 };
+
+// Head h's sink in the units of the log-sum-exps (times log2 e), minus infinity without one: 2^(-inf) = 0.
+__device__ __forceinline__ float sink_log2(const Extras& ex, int h) { return ex.sinks ? ex.sinks[h] * LOG2_E : -INFINITY; }
 
 // The keys a token at position kv_len - 1 sees are numbered consecutively: the window's keys keep their
 // positions, the kept first tokens that lie before the window take the numbers just below it.
@@ -76,10 +83,10 @@ constexpr int THREADS = WARPS * 32;
 template <int D>
 __device__ __forceinline__ void merge_row(const float* __restrict__ mid_o, const float* __restrict__ lse,
                                           int num_splits, bf16* __restrict__ out_row, int first, int step,
-                                          float sink_log2, const bf16* __restrict__ gate_row) {
+                                          float sink, const bf16* __restrict__ gate_row) {
   float mx = -INFINITY;
   for (int s = 0; s < num_splits; ++s) mx = fmaxf(mx, __ldcg(lse + s));
-  const float sink_w = exp2f(sink_log2 - mx);  // no sink: 2^(-inf) = 0
+  const float sink_w = exp2f(sink - mx);  // no sink: 2^(-inf) = 0
   for (int d = 4 * first; d < D; d += 4 * step) {
     float acc[4] = {0.f, 0.f, 0.f, 0.f};
     float wsum = sink_w;
@@ -136,12 +143,12 @@ __device__ __forceinline__ bool drew_last_ticket(int* ticket, int num_splits) {
 template <int D>
 __device__ __forceinline__ void merge_pair(const float* __restrict__ mid_o, const float* __restrict__ mid_lse,
                                            long first_head, int G, int num_splits, int slices,
-                                           bf16* __restrict__ out_rows, float sink_log2 = -INFINITY,
-                                           const bf16* __restrict__ gate_rows = nullptr) {
+                                           bf16* __restrict__ out_rows, const Extras& ex, int kv_head_first,
+                                           const bf16* __restrict__ gate_rows) {
   constexpr int PER_ROW = D / 4 < 32 ? D / 4 : 32;  // threads on one row, 4 values each
   for (int g = threadIdx.x / PER_ROW; g < G; g += THREADS / PER_ROW)
     merge_row<D>(mid_o + (first_head + g) * num_splits * D, mid_lse + (first_head + g) * num_splits, slices,
-                 out_rows + (long)g * D, threadIdx.x % PER_ROW, PER_ROW, sink_log2,
+                 out_rows + (long)g * D, threadIdx.x % PER_ROW, PER_ROW, sink_log2(ex, kv_head_first + g),
                  gate_rows ? gate_rows + (long)g * D : nullptr);
 }
 
@@ -232,7 +239,7 @@ decode_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* kp
       pdl_launch_dependents();
       if (drew_last_ticket(ticket, slices))
         merge_pair<D>(mid_o, mid_lse, (long)slot * nq + kvh * G, G, num_splits, slices,
-                      out + ((long)tok * nq + kvh * G) * D, ex.sink_log2, gate_rows);
+                      out + ((long)tok * nq + kvh * G) * D, ex, kvh * G, gate_rows);
     }
     return;
   }
@@ -351,6 +358,24 @@ decode_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* kp
         }
         if (rotate)
           rotate_chunks(a, b, nt.cos_t + (long)p * HALF, nt.sin_t + (long)p * HALF, c, HALF, nt.pairing);
+        if (is_q && nt.q_scale) {
+          const float f = nt.q_scale[tok];
+#pragma unroll
+          for (int e = 0; e < 8; ++e) {
+            a[e] *= f;
+            b[e] *= f;
+          }
+        }
+      } else if (nt.v_first) {
+        const bf16* first = nt.v_first + (long)tok * nt.v_first_stride + (long)kvh * D;
+        float fa[8], fb[8];
+        load8(first + 8 * c, fa);
+        load8(first + HALF + 8 * c, fb);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          a[e] = (1.f - nt.v_share) * a[e] + nt.v_share * fa[e];
+          b[e] = (1.f - nt.v_share) * b[e] + nt.v_share * fb[e];
+        }
       }
       if (is_q) {
         store8(reinterpret_cast<bf16*>(q_s + swz<D>(item, c)), a);
@@ -520,7 +545,7 @@ decode_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* kp
     }
     const int head = kvh * G + g;
     if (slices == 1) {
-      float val = acc / (l + exp2f(ex.sink_log2 - m * scale_log2));
+      float val = acc / (l + exp2f(sink_log2(ex, head) - m * scale_log2));
       if (gate_rows) val *= 1.f / (1.f + __expf(-__bfloat162float(gate_rows[(long)g * D + d])));
       out[((long)tok * nq + head) * D + d] = __float2bfloat16_rn(val);
     } else {
@@ -530,7 +555,7 @@ decode_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* kp
   }
   if (ticket && drew_last_ticket(ticket, slices))
     merge_pair<D>(mid_o, mid_lse, (long)slot * nq + kvh * G, G, num_splits, slices,
-                  out + ((long)tok * nq + kvh * G) * D, ex.sink_log2, gate_rows);
+                  out + ((long)tok * nq + kvh * G) * D, ex, kvh * G, gate_rows);
 }
 
 // The merge as a kernel of its own: one block per (kv head, sequence).
@@ -552,7 +577,7 @@ decode_combine_kernel(const float* __restrict__ mid_o, const float* __restrict__
                                longest_len, ex.keep);
   if (slices == 1) return;  // a sequence in one slice: its block wrote the result itself
   merge_pair<D>(mid_o, mid_lse, (long)slot * nq + kvh * G, G, num_splits, slices,
-                out + ((long)tok * nq + kvh * G) * D, ex.sink_log2,
+                out + ((long)tok * nq + kvh * G) * D, ex, kvh * G,
                 ex.gate ? ex.gate + (long)tok * ex.gate_stride + (long)kvh * G * D : nullptr);
 }
 
@@ -661,21 +686,21 @@ Q3_EXPORT int q3_paged_attention_decode(const void* q, int q_stride, const void*
                                 nullptr, tickets, longest_len, stream);
 }
 
-// The same with a window that keeps the sequence's first `keep_first` tokens, a sink (a score without a
-// value in the softmax's denominator; has_sink 0: none) and a gate (null, or rows of gate_stride values of
+// The same with a window that keeps the sequence's first `keep_first` tokens, sinks (null, or per head, fp32
+// [nq], a score without a value in the softmax's denominator) and a gate (null, or rows of gate_stride values of
 // which the first nq * D gate the heads' outputs by their sigmoid; 16-byte alignment is not needed).
 Q3_EXPORT int q3_paged_attention_decode_sink(const void* q, int q_stride, const void* kpages, const void* vpages,
                                              const int* block_table, int max_pages, const int* kv_lens,
                                              const int* cu_seqlens, const int* seq_list, void* out, float* mid_o,
                                              float* mid_lse, int num_seqs, int nq, int nkv, int D, int ps,
                                              float scale, int window, int num_splits, int* tickets,
-                                             const int* longest_len, int keep_first, int has_sink, float sink,
+                                             const int* longest_len, int keep_first, const float* sinks,
                                              const void* gate, int gate_stride, float softcap, cudaStream_t stream) {
   if (keep_first < 0 || (gate && gate_stride < nq * D) || softcap < 0.f || !(scale > 0.f)) return Q3_ERR_ARGUMENT;
   Extras ex;
   ex.cap_raw = softcap / scale;
   ex.keep = window > 0 ? keep_first : 0;
-  ex.sink_log2 = has_sink ? sink * 1.4426950408889634f : -INFINITY;
+  ex.sinks = sinks;
   ex.gate = (const bf16*)gate;
   ex.gate_stride = gate_stride;
   return dispatch_decode<false>(q, q_stride, kpages, vpages, block_table, max_pages, kv_lens, cu_seqlens, seq_list,
@@ -690,9 +715,11 @@ Q3_EXPORT int q3_paged_attention_decode_sink(const void* q, int q_stride, const 
 // null.  The key and value of the newest token are written to their pages; q is not written
 // back.  `error_word` (may be null) is set to Q3_ERR_POSITION if a newest position lies beyond
 // the tables; that token is then left unrotated and the result is invalid.
-// (keep_first, has_sink, sink, gate, gate_stride, softcap: as in q3_paged_attention_decode_sink; softcap: scores
+// (keep_first, sinks, gate, gate_stride, softcap: as in q3_paged_attention_decode_sink; softcap: scores
 // become softcap * tanh(score / softcap) after the scale, 0 for none.  v_from_k: rows hold nq + nkv heads only and
-// a key head as projected is also its value.)
+// a key head as projected is also its value.  q_scale: null, or fp32, one factor per packed token for its queries,
+// after norm and rotation.  v_first: null, or bf16 rows, v_first_stride apart per packed token, with nkv heads of D:
+// the token's value becomes (1 - v_share) * its own + v_share * v_first's, in fp32, rounded once.)
 Q3_EXPORT int q3_paged_attention_decode_fused_sink(const void* qkv, int q_stride, void* kpages, void* vpages,
                                                    const int* block_table, int max_pages, const int* kv_lens,
                                                    const int* cu_seqlens, const int* seq_list, void* out,
@@ -700,19 +727,23 @@ Q3_EXPORT int q3_paged_attention_decode_fused_sink(const void* qkv, int q_stride
                                                    int ps, float scale, int window, int num_splits, const float* q_w,
                                                    const float* k_w, float eps, const float* cos_t,
                                                    const float* sin_t, int max_pos, int pairing, int* error_word,
-                                                   int* tickets, const int* longest_len, int keep_first, int has_sink,
-                                                   float sink, const void* gate, int gate_stride, float softcap,
-                                                   int v_from_k, cudaStream_t stream) {
+                                                   int* tickets, const int* longest_len, int keep_first,
+                                                   const float* sinks, const void* gate, int gate_stride, float softcap,
+                                                   int v_from_k, const float* q_scale, const void* v_first,
+                                                   int v_first_stride, float v_share, cudaStream_t stream) {
   if ((cos_t && (!sin_t || max_pos < 1)) || (!q_w) != (!k_w) || pairing < 0 || pairing > 1) return Q3_ERR_ARGUMENT;
   if (keep_first < 0 || (gate && gate_stride < nq * D) || softcap < 0.f || !(scale > 0.f)) return Q3_ERR_ARGUMENT;
   const uintptr_t bits = (uintptr_t)qkv | (uintptr_t)kpages | (uintptr_t)vpages | (uintptr_t)q_w | (uintptr_t)k_w |
                          (uintptr_t)cos_t | (uintptr_t)sin_t;
   if (bits & 15) return Q3_ERR_UNSUPPORTED;
-  NewToken nt{q_w, k_w, cos_t, sin_t, (bf16*)kpages, (bf16*)vpages, eps, max_pos, pairing, v_from_k ? 1 : 0};
+  if (v_first && (v_from_k || v_first_stride < nkv * D)) return Q3_ERR_ARGUMENT;
+  if (v_first && (v_first_stride % 8 || ((uintptr_t)v_first & 15))) return Q3_ERR_UNSUPPORTED;
+  NewToken nt{q_w, k_w, cos_t, sin_t, (bf16*)kpages, (bf16*)vpages, eps, max_pos, pairing, v_from_k ? 1 : 0,
+              q_scale, (const bf16*)v_first, v_first_stride, v_share};
   Extras ex;
   ex.cap_raw = softcap / scale;
   ex.keep = window > 0 ? keep_first : 0;
-  ex.sink_log2 = has_sink ? sink * 1.4426950408889634f : -INFINITY;
+  ex.sinks = sinks;
   ex.gate = (const bf16*)gate;
   ex.gate_stride = gate_stride;
   return dispatch_decode<true>(qkv, q_stride, kpages, vpages, block_table, max_pages, kv_lens, cu_seqlens, seq_list,
@@ -731,7 +762,8 @@ Q3_EXPORT int q3_paged_attention_decode_fused(const void* qkv, int q_stride, voi
   return q3_paged_attention_decode_fused_sink(qkv, q_stride, kpages, vpages, block_table, max_pages, kv_lens,
                                               cu_seqlens, seq_list, out, mid_o, mid_lse, num_seqs, nq, nkv, D, ps, scale,
                                               window, num_splits, q_w, k_w, eps, cos_t, sin_t, max_pos, pairing,
-                                              error_word, tickets, longest_len, 0, 0, 0.f, nullptr, 0, 0.f, 0, stream);
+                                              error_word, tickets, longest_len, 0, nullptr, nullptr, 0, 0.f, 0, nullptr,
+                                              nullptr, 0, 0.f, stream);
 }
 
 // ---------------------------------------------------------------------------------------------

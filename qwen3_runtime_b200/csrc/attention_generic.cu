@@ -3,8 +3,8 @@
 // 16-byte loads), a value size of its own up to 256, any head counts, any page size, optional
 // window), used by the fp32 path and wherever a specialised kernel refuses a size.  Options: a
 // window that leaves the sequence's first `keep_first` keys readable (they are visited first, in
-// tiles of their own, then the window's); a sink, one more score without a value in the softmax's
-// denominator, p_j = exp(s_j) / (exp(sink) + sum exp(s_j')); a gate, the result times
+// tiles of their own, then the window's); sinks, per head one more score without a value in the softmax's
+// denominator, p_j = exp(s_j) / (exp(sink_h) + sum exp(s_j')); a gate, the result times
 // sigmoid(gate[t, h, d]) before the one rounding; a chunked mask (`chunk` > 0: position p reads keys from
 // floor(p / chunk) * chunk on, chunks counted from the sequence's position 0); capped scores
 // (`softcap` > 0: s <- softcap * tanh(s / softcap) after the scale).  A second kernel is differential
@@ -27,7 +27,7 @@ __global__ void paged_attention_generic_kernel(const T* __restrict__ q, int q_st
                                                const int* __restrict__ token_seq,
                                                const int* __restrict__ positions, T* __restrict__ out,
                                                long out_stride, int num_tokens, int nq, int nkv, int D, int Dv, int ps, float scale,
-                                               int window, int keep_first, int has_sink, float sink,
+                                               int window, int keep_first, const float* __restrict__ sinks,
                                                const T* __restrict__ gate, long gate_stride, int chunk,
                                                float softcap, const float* __restrict__ turns, int turn_pairs,
                                                int turn_pairing) {
@@ -99,7 +99,8 @@ __global__ void paged_attention_generic_kernel(const T* __restrict__ q, int q_st
     }
   }
   T* orow = out + (long)t * out_stride + (long)h * Dv;
-  if (has_sink) {  // one more score in the denominator
+  if (sinks) {  // one more score in the denominator
+    const float sink = sinks[h];
     const float m_all = fmaxf(m, sink), corr = expf(m - m_all);
     l = l * corr + expf(sink - m_all);
 #pragma unroll
@@ -137,7 +138,8 @@ __global__ void paged_attention_generic_kernel(const T* __restrict__ q, int q_st
 
 // q: [num_tokens, *] with row stride q_stride (elements), head h at column h*D.  Keys are
 // [pages, nkv, ps, D], values [pages, nkv, ps, Dv].  out: rows out_stride elements apart, head h at
-// column h*Dv.  window <= 0: none; keep_first counts only with a window; gate: rows gate_stride elements
+// column h*Dv.  window <= 0: none; keep_first counts only with a window; sinks: fp32
+// [nq] scores without a value, or null; gate: rows gate_stride elements
 // apart, head h at column h*Dv, or null.  chunk <= 0: no chunked mask; softcap <= 0: scores as they are.
 // turns: null, or fp32 [num_tokens, 2, turn_pairs] (cos, then sin): the values in the cache are turned by their own
 // positions and a head's result is turned back by the token's angles (pairs (m, m + turn_pairs), or with
@@ -146,7 +148,7 @@ Q3_EXPORT int q3_paged_attention_generic(int dtype, const void* q, int q_stride,
                                          const void* vpages, const int* block_table, int max_pages,
                                          const int* token_seq, const int* positions, void* out,
                                          long out_stride, int num_tokens, int nq, int nkv, int D, int Dv, int ps,
-                                         float scale, int window, int keep_first, int has_sink, float sink,
+                                         float scale, int window, int keep_first, const float* sinks,
                                          const void* gate, long gate_stride, int chunk, float softcap,
                                          const float* turns, int turn_pairs, int turn_pairing, cudaStream_t stream) {
   if (!q || !kpages || !vpages || !block_table || !token_seq || !positions || !out) return Q3_ERR_ARGUMENT;
@@ -165,12 +167,12 @@ Q3_EXPORT int q3_paged_attention_generic(int dtype, const void* q, int q_stride,
     paged_attention_generic_kernel<float, WARPS><<<blocks, WARPS * 32, smem, stream>>>(
         (const float*)q, q_stride, (const float*)kpages, (const float*)vpages, block_table, max_pages,
         token_seq, positions, (float*)out, out_stride, num_tokens, nq, nkv, D, Dv, ps, scale, window, keep_first,
-        has_sink, sink, (const float*)gate, gate_stride, chunk, softcap, turns, turn_pairs, turn_pairing);
+        sinks, (const float*)gate, gate_stride, chunk, softcap, turns, turn_pairs, turn_pairing);
   else if (dtype == Q3_DTYPE_BF16)
     paged_attention_generic_kernel<bf16, WARPS><<<blocks, WARPS * 32, smem, stream>>>(
         (const bf16*)q, q_stride, (const bf16*)kpages, (const bf16*)vpages, block_table, max_pages,
         token_seq, positions, (bf16*)out, out_stride, num_tokens, nq, nkv, D, Dv, ps, scale, window, keep_first,
-        has_sink, sink, (const bf16*)gate, gate_stride, chunk, softcap, turns, turn_pairs, turn_pairing);
+        sinks, (const bf16*)gate, gate_stride, chunk, softcap, turns, turn_pairs, turn_pairing);
   else
     return Q3_ERR_ARGUMENT;
   return q3_launch_status();

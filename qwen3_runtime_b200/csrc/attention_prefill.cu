@@ -11,8 +11,8 @@
 // max(0, p - window + 1) .. p; p = kv_len - q_len + its index in the portion
 // (attention/pytorch.py:12-15).  Keys the block does not need are zero-filled, never read.
 // Optional: with a window the sequence's first `keep` tokens stay visible (their tiles come before the
-// window's); a sink, a score without a value that joins the softmax's denominator (sink_log2 = score *
-// log2 e, minus infinity for none); a gate whose sigmoid multiplies the result.
+// window's); sinks, per head a score without a value that joins the softmax's denominator;
+// a gate whose sigmoid multiplies the result.
 //
 // The block finds its work item by walking cu_seqlens (sequences with one token can be left
 // to the decode kernel: skip_single).
@@ -33,7 +33,7 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* _
                          const bf16* __restrict__ vpages, const int* __restrict__ block_table, int max_pages,
                          const int* __restrict__ kv_lens, const int* __restrict__ cu_seqlens,
                          bf16* __restrict__ out, int num_seqs, int nq, int nkv, int ps, float scale_log2,
-                         int window, int skip_single, int keep, float sink_log2, const bf16* __restrict__ gate,
+                         int window, int skip_single, int keep, const float* __restrict__ sinks, const bf16* __restrict__ gate,
                          int gate_stride, float cap_raw) {
   constexpr int CHUNKS = D / 8;
   constexpr int TILE_BYTES = TILE * D * 2;
@@ -259,7 +259,8 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* _
     const int R = row0 + warp * 16 + (lane >> 2) + r * 8;
     if (R >= rows) continue;
     const int tk = R / G, hd = kvh * G + (R - tk * G);
-    const float inv = 1.f / (l_run[r] + exp2f(sink_log2 - m_run[r] * scale_log2));  // no sink: 2^(-inf) = 0
+    if (sinks) l_run[r] += exp2f(sinks[hd] * LOG2_E - m_run[r] * scale_log2);
+    const float inv = 1.f / l_run[r];
     bf16* dst = out + ((long)(tok0 + tk) * nq + hd) * D + 2 * (lane & 3);
     if (gate) {
       const bf16* g = gate + (long)(tok0 + tk) * gate_stride + (long)hd * D + 2 * (lane & 3);
@@ -280,7 +281,7 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* _
 template <int D>
 int launch_prefill(const bf16* q, int q_stride, const bf16* kpages, const bf16* vpages, const int* block_table,
                    int max_pages, const int* kv_lens, const int* cu_seqlens, bf16* out, int num_seqs, int num_work,
-                   int nq, int nkv, int ps, float scale, int window, int skip_single, int keep, float sink_log2,
+                   int nq, int nkv, int ps, float scale, int window, int skip_single, int keep, const float* sinks,
                    const bf16* gate, int gate_stride, float softcap, cudaStream_t stream) {
   const size_t smem = (size_t)BLOCK_M * D * 2 + (size_t)STAGES * 2 * TILE * D * 2;
   static bool configured_on[Q3_MAX_DEVICES];
@@ -295,7 +296,7 @@ int launch_prefill(const bf16* q, int q_stride, const bf16* kpages, const bf16* 
   prefill_attention_kernel<D><<<grid, THREADS, smem, stream>>>(q, q_stride, kpages, vpages, block_table, max_pages,
                                                                kv_lens, cu_seqlens, out, num_seqs, nq, nkv, ps,
                                                                scale * 1.4426950408889634f, window, skip_single,
-                                                               keep, sink_log2, gate, gate_stride, softcap / scale);
+                                                               keep, sinks, gate, gate_stride, softcap / scale);
   return q3_launch_status();
 }
 
@@ -304,15 +305,15 @@ int launch_prefill(const bf16* q, int q_stride, const bf16* kpages, const bf16* 
 // num_work = sum over the sequences this launch serves of ceil(q_len * (nq / nkv) / 128).
 // head_dim 64 or 128; bfloat16 only.  With skip_single, sequences of one token are left out
 // (their rows of `out` are not written).
-// keep_first: with a window, the sequence's first tokens stay visible.  has_sink / sink: a score without a
-// value in the softmax's denominator.  gate: null, or rows of gate_stride values of which the first nq * D
+// keep_first: with a window, the sequence's first tokens stay visible.  sinks: null, or per head (fp32 [nq]) a
+// score without a value in the softmax's denominator.  gate: null, or rows of gate_stride values of which the first nq * D
 // gate the heads' outputs by their sigmoid.  softcap: scores become softcap * tanh(score / softcap) after the
 // scale; 0 for none.
 Q3_EXPORT int q3_paged_attention_prefill_sink(const void* q, int q_stride, const void* kpages, const void* vpages,
                                               const int* block_table, int max_pages, const int* kv_lens,
                                               const int* cu_seqlens, void* out, int num_seqs, int num_work, int nq,
                                               int nkv, int D, int ps, float scale, int window, int skip_single,
-                                              int keep_first, int has_sink, float sink, const void* gate,
+                                              int keep_first, const float* sinks, const void* gate,
                                               int gate_stride, float softcap, cudaStream_t stream) {
   if (!q || !kpages || !vpages || !block_table || !kv_lens || !cu_seqlens || !out) return Q3_ERR_ARGUMENT;
   if (nq < 1 || nkv < 1 || nq % nkv || ps < 1 || num_seqs < 0 || num_work < 0) return Q3_ERR_ARGUMENT;
@@ -320,15 +321,14 @@ Q3_EXPORT int q3_paged_attention_prefill_sink(const void* q, int q_stride, const
   if (q_stride % 8 || nkv > 65535) return Q3_ERR_UNSUPPORTED;
   if (num_work == 0) return Q3_OK;
   const int keep = window > 0 ? keep_first : 0;
-  const float sink_log2 = has_sink ? sink * 1.4426950408889634f : -INFINITY;
   if (D == 64)
     return launch_prefill<64>((const bf16*)q, q_stride, (const bf16*)kpages, (const bf16*)vpages, block_table,
                               max_pages, kv_lens, cu_seqlens, (bf16*)out, num_seqs, num_work, nq, nkv, ps, scale,
-                              window, skip_single, keep, sink_log2, (const bf16*)gate, gate_stride, softcap, stream);
+                              window, skip_single, keep, sinks, (const bf16*)gate, gate_stride, softcap, stream);
   if (D == 128)
     return launch_prefill<128>((const bf16*)q, q_stride, (const bf16*)kpages, (const bf16*)vpages, block_table,
                                max_pages, kv_lens, cu_seqlens, (bf16*)out, num_seqs, num_work, nq, nkv, ps, scale,
-                               window, skip_single, keep, sink_log2, (const bf16*)gate, gate_stride, softcap, stream);
+                               window, skip_single, keep, sinks, (const bf16*)gate, gate_stride, softcap, stream);
   return Q3_ERR_UNSUPPORTED;
 }
 
@@ -338,6 +338,6 @@ Q3_EXPORT int q3_paged_attention_prefill(const void* q, int q_stride, const void
                                          int nkv, int D, int ps, float scale, int window, int skip_single,
                                          cudaStream_t stream) {
   return q3_paged_attention_prefill_sink(q, q_stride, kpages, vpages, block_table, max_pages, kv_lens, cu_seqlens, out,
-                                         num_seqs, num_work, nq, nkv, D, ps, scale, window, skip_single, 0, 0, 0.f,
+                                         num_seqs, num_work, nq, nkv, D, ps, scale, window, skip_single, 0, nullptr,
                                          nullptr, 0, 0.f, stream);
 }

@@ -1,8 +1,8 @@
 // Causal attention of prompt portions over the paged cache on the 5th-generation tensor
 // cores: S = Q K^T and O += P V are tcgen05.mma with accumulators in tensor memory, Q, K and V
 // tiles arrive by TMA (128-byte swizzle) straight from the QKV buffer and the cache pages.
-// bfloat16, head_dim 128, group size a divisor of 128, page size 8/16/32/64, no window (a chunked mask
-// and turned values are options); the mma.sync kernels serve everything else.
+// bfloat16, head_dim 128, group size a divisor of 128, page size 8/16/32/64, no window (a chunked mask,
+// turned values and sinks are options); the mma.sync kernels serve everything else.
 //
 // Work item: (sequence, kv head, two consecutive blocks of 128 rows, A and B); rows are the
 // (query token, head of the group) pairs in token-major order, so one 3-D TMA box
@@ -68,7 +68,7 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
                             int max_pages, const int* __restrict__ kv_lens, const int* __restrict__ cu_seqlens,
                             bf16* __restrict__ out, int num_seqs, int num_work, int nq, int nkv, int ps,
                             float scale_log2, int skip_single, int chunk, const float* __restrict__ turns,
-                            int* __restrict__ error_word) {
+                            const float* __restrict__ sinks, int* __restrict__ error_word) {
   extern __shared__ unsigned char smem_raw[];
   unsigned char* base = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~(uintptr_t)1023);
   unsigned char* q_s = base;                         // 2 blocks x [2 halves][128 rows][128 B]
@@ -393,6 +393,8 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
       if (ok && my_tiles) ok = mbar_wait(bar(BAR_PV_FULL + x), (my_tiles - 1) & 1, &abort_flag);
       if (ok && my_tiles) {
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        // a head's sink: one more term in the denominator, in the units of the row's reference point
+        if (sinks && row_ok) l_run += exp2f(sinks[kvh * G + R % G] * LOG2_E - m_ref * scale_log2);
         const float inv = 1.f / l_run;
         bf16* dst = row_ok ? out + ((long)(tok0 + R / G) * nq + kvh * G + R % G) * D : nullptr;
         if (turns) {  // turned values: the sum is turned back, element c with element c + D / 2
@@ -457,13 +459,14 @@ prefill_attention_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __
 // Returns Q3_ERR_UNSUPPORTED for shapes this kernel does not take (the caller then uses the
 // mma.sync kernel).  chunk > 0: a token sees the keys of its own chunk of that many tokens only.  turns: null, or
 // fp32 [num_tokens, 2, 64], cos then sin per pair (m, m + 64): the cached values are turned by their positions and a
-// head's result is turned back by its token's angles.  error_word: device int set to 2 if a wait inside the kernel expired.
+// head's result is turned back by its token's angles.  sinks: null, or fp32 [nq], per head a score without a value in the
+// softmax's denominator.  error_word: device int set to 2 if a wait inside the kernel expired.
 Q3_EXPORT int q3_paged_attention_prefill_tc(const void* q, int q_stride, int num_tokens, const void* kpages,
                                             const void* vpages, long num_rows_kv, const int* block_table,
                                             int max_pages, const int* kv_lens, const int* cu_seqlens, void* out,
                                             int num_seqs, int num_work, int nq, int nkv, int head_dim, int ps,
                                             float scale, int skip_single, int chunk, const float* turns,
-                                            int* error_word, cudaStream_t stream) {
+                                            const float* sinks, int* error_word, cudaStream_t stream) {
   if (chunk < 0 || ((uintptr_t)turns & 15)) return Q3_ERR_ARGUMENT;
   if (!q || !kpages || !vpages || !block_table || !kv_lens || !cu_seqlens || !out) return Q3_ERR_ARGUMENT;
   if (nq < 1 || nkv < 1 || nq % nkv) return Q3_ERR_ARGUMENT;
@@ -501,6 +504,6 @@ Q3_EXPORT int q3_paged_attention_prefill_tc(const void* q, int q_stride, int num
   prefill_attention_tc_kernel<<<grid, THREADS, SMEM_BYTES, stream>>>(tq, tk, tv, block_table, max_pages, kv_lens,
                                                                     cu_seqlens, (bf16*)out, num_seqs, num_work, nq,
                                                                     nkv, ps, scale * 1.4426950408889634f,
-                                                                    skip_single, chunk, turns, error_word);
+                                                                    skip_single, chunk, turns, sinks, error_word);
   return q3_launch_status();
 }

@@ -38,6 +38,15 @@ template <typename T> __device__ __forceinline__ T from_f32(float x);
 template <> __device__ __forceinline__ float from_f32<float>(float x) { return x; }
 template <> __device__ __forceinline__ bf16 from_f32<bf16>(float x) { return __float2bfloat16_rn(x); }
 
+constexpr float LOG2_E = 1.4426950408889634f;
+
+// The unit of a gated feed-forward: act 0 silu(g) * u, act 1 gelu(g) * u in gelu's tanh form, which is
+// g * sigmoid(2 y), y = sqrt(2 / pi) (g + 0.044715 g^3), since (1 + tanh y) / 2 = sigmoid(2 y).
+__device__ __forceinline__ float gated_unit(float g, float u, int act) {
+  const float y = act ? 1.5957691216057308f * (g + 0.044715f * g * g * g) : g;
+  return (g / (1.f + expf(-y))) * u;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -82,9 +82,9 @@ route_logits_kernel(const T* __restrict__ h, long h_stride, const float* __restr
 }
 
 // mode 0: weights are the chosen logits' sigmoids; 1: those divided by their sum; 2: the softmax over
-// the chosen logits only.
+// the chosen logits only; all times `scale`.
 __global__ void route_pick_kernel(float* __restrict__ logits, int num_tokens, int E, int top, int mode,
-                                  int* __restrict__ chosen, float* __restrict__ weights) {
+                                  float scale, int* __restrict__ chosen, float* __restrict__ weights) {
   pdl_wait();
   pdl_launch_dependents();
   const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -120,17 +120,20 @@ __global__ void route_pick_kernel(float* __restrict__ logits, int num_tokens, in
     total += score;
     __syncwarp();
   }
-  if (mode)
-    for (int k = lane; k < top; k += 32) weights[(long)t * top + k] /= total;
+  if (mode || scale != 1.f)
+    for (int k = lane; k < top; k += 32) {
+      const float w = weights[(long)t * top + k];
+      weights[(long)t * top + k] = (mode ? w / total : w) * scale;
+    }
 }
 
 // mode 3: s = softmax over all E logits; the choice is made on c = s + correction (correction null: on s)
 // among the outputs of the `keep` best of `count` equal groups of neighbours (a group's score: its largest
 // c; count <= 1: no groups), lowest index on a tie; the weights are the chosen s, divided by their sum +
-// 1e-20 when `renorm`.  One warp per token; c and the groups' scores wait in shared memory.
+// 1e-20 when `renorm`, times `scale`.  One warp per token; c and the groups' scores wait in shared memory.
 __global__ void route_pick_softmax_all_kernel(const float* __restrict__ logits, int num_tokens, int E, int top,
                                               const float* __restrict__ correction, int count, int keep, int renorm,
-                                              int* __restrict__ chosen, float* __restrict__ weights) {
+                                              float scale, int* __restrict__ chosen, float* __restrict__ weights) {
   extern __shared__ float pick_smem[];  // per warp: c[E], group scores[count]
   pdl_wait();
   pdl_launch_dependents();
@@ -197,15 +200,18 @@ __global__ void route_pick_softmax_all_kernel(const float* __restrict__ logits, 
     total += score;
     __syncwarp();
   }
-  if (renorm)
-    for (int k = lane; k < top; k += 32) weights[(long)t * top + k] /= total + 1e-20f;
+  if (renorm || scale != 1.f)
+    for (int k = lane; k < top; k += 32) {
+      const float w = weights[(long)t * top + k];
+      weights[(long)t * top + k] = (renorm ? w / (total + 1e-20f) : w) * scale;
+    }
 }
 
 // logits: fp32 scratch [num_tokens, E] (left with the chosen entries at -inf).
-// mode 3 takes correction (fp32 [E] or null), count and keep (groups) and renorm; the other modes ignore them.
+// scale: a factor on all weights.  mode 3 takes correction (fp32 [E] or null), count and keep (groups) and renorm; the other modes ignore them.
 Q3_EXPORT int q3_route_top(int dtype, const void* h, long h_stride, const float* router, int num_tokens, int E, int W,
                            int top, int mode, float* logits, int* chosen, float* weights, const float* correction,
-                           int count, int keep, int renorm, cudaStream_t stream) {
+                           int count, int keep, int renorm, float scale, cudaStream_t stream) {
   if (!h || !router || !logits || !chosen || !weights || E < 1 || W < 1 || top < 1 || top > E) return Q3_ERR_ARGUMENT;
   if (mode == 3 && count > 1 && (E % count || keep < 1 || keep > count || top > keep * (E / count)))
     return Q3_ERR_ARGUMENT;
@@ -234,11 +240,11 @@ Q3_EXPORT int q3_route_top(int dtype, const void* h, long h_stride, const float*
     const size_t pick = (size_t)4 * (E + (count > 1 ? count : 0)) * sizeof(float);
     if (pick > 48 * 1024) return Q3_ERR_UNSUPPORTED;
     e = launch_pdl(route_pick_softmax_all_kernel, dim3((num_tokens + 3) / 4), dim3(128), pick, stream,
-                   (const float*)logits, num_tokens, E, top, correction, count, keep, renorm, chosen, weights);
+                   (const float*)logits, num_tokens, E, top, correction, count, keep, renorm, scale, chosen, weights);
     return e == cudaSuccess ? Q3_OK : Q3_ERR_LAUNCH;
   }
   e = launch_pdl(route_pick_kernel, dim3((num_tokens + 3) / 4), dim3(128), 0, stream, logits, num_tokens, E, top,
-                 mode, chosen, weights);
+                 mode, scale, chosen, weights);
   return e == cudaSuccess ? Q3_OK : Q3_ERR_LAUNCH;
 }
 

@@ -45,7 +45,7 @@ template <int NT, int MODE, int WARPS_, int MINB_>
 __global__ void __launch_bounds__(WARPS_ * 32, MINB_)
 gemm_small_m_kernel(const bf16* __restrict__ x, int ldx, const bf16* __restrict__ W, int ldw,
                     void* __restrict__ out, int ldo, int M, int N, int K, int KS, int kper, int up_offset,
-                    int prefetch_l2) {
+                    int act, int prefetch_l2) {
   constexpr int SETS = MODE == OUT_SWIGLU ? 2 : 1;
   constexpr int U = 2;  // k-blocks of 32 in flight per thread (64 registers: many warps instead)
   __shared__ float red[MAX_WARPS][SETS * NT * 4][32];
@@ -157,7 +157,7 @@ gemm_small_m_kernel(const bf16* __restrict__ x, int ldx, const bf16* __restrict_
       const int token = n * 8 + 2 * t + (e & 1);
       if (feature >= N || token >= M) continue;
       float v = acc[0][n][e];
-      if (MODE == OUT_SWIGLU) v = (v / (1.f + expf(-v))) * acc[SETS - 1][n][e];
+      if (MODE == OUT_SWIGLU) v = gated_unit(v, acc[SETS - 1][n][e], act);
       if (MODE == OUT_F32)
         reinterpret_cast<float*>(out)[(long)token * ldo + feature] = v;
       else
@@ -167,7 +167,7 @@ gemm_small_m_kernel(const bf16* __restrict__ x, int ldx, const bf16* __restrict_
 
 template <int NT, int MODE>
 int launch(const bf16* x, int ldx, const bf16* W, int ldw, void* out, int ldo, int M, int N, int K, int up_offset,
-           cudaStream_t stream) {
+           int act, cudaStream_t stream) {
   const int tiles = (N + 15) / 16;
   // split K until there are about 16 warps per SM, but keep slices of at least 256
   int KS = 1;
@@ -181,17 +181,18 @@ int launch(const bf16* x, int ldx, const bf16* W, int ldw, void* out, int ldo, i
   const int prefetch_l2 = (long)N * K * 2 * (MODE == OUT_SWIGLU ? 2 : 1) <= (64L << 20);
   if (warps == 16)
     err = launch_pdl(gemm_small_m_kernel<NT, MODE, 16, 2>, dim3(blocks), dim3(512), 0, stream, x, ldx, W, ldw, out,
-                     ldo, M, N, K, KS, kper, up_offset, prefetch_l2);
+                     ldo, M, N, K, KS, kper, up_offset, act, prefetch_l2);
   else
     err = launch_pdl(gemm_small_m_kernel<NT, MODE, 8, 4>, dim3(blocks), dim3(256), 0, stream, x, ldx, W, ldw, out,
-                     ldo, M, N, K, KS, kper, up_offset, prefetch_l2);
+                     ldo, M, N, K, KS, kper, up_offset, act, prefetch_l2);
   return err == cudaSuccess ? Q3_OK : Q3_ERR_LAUNCH;
 }
 
 }  // namespace
 
 // mode 0: out bf16 [M, N]; 1: out fp32 [M, N]; 2: W is [2 * N, K] with gate rows first and up
-// rows from row `N`, out bf16 [M, N] = silu(x W_gate^T) * (x W_up^T).
+// rows from row `N`, out bf16 [M, N] = silu(x W_gate^T) * (x W_up^T); 3: the same with gelu (tanh form)
+// in place of silu.
 // M <= 16; K a multiple of 8; leading dimensions in elements (ldx, ldw multiples of 8).
 Q3_EXPORT int q3_gemm_small_m(int mode, const void* x, int ldx, const void* W, int ldw, void* out, int ldo, int M,
                               int N, int K, cudaStream_t stream) {
@@ -199,9 +200,11 @@ Q3_EXPORT int q3_gemm_small_m(int mode, const void* x, int ldx, const void* W, i
   if (M > 16 || K % 8 || ldx % 8 || ldw % 8 || ldx < K || ldw < K || ldo < N) return Q3_ERR_UNSUPPORTED;
   if (((uintptr_t)x | (uintptr_t)W) & 15) return Q3_ERR_UNSUPPORTED;
   if (M == 0) return Q3_OK;
+  const int act = mode == 3;
+  if (act) mode = OUT_SWIGLU;
   const bf16* xp = (const bf16*)x;
   const bf16* wp = (const bf16*)W;
-#define Q3_GEMM_CASE(NT, MODE) return launch<NT, MODE>(xp, ldx, wp, ldw, out, ldo, M, N, K, mode == 2 ? N : 0, stream)
+#define Q3_GEMM_CASE(NT, MODE) return launch<NT, MODE>(xp, ldx, wp, ldw, out, ldo, M, N, K, mode == OUT_SWIGLU ? N : 0, act, stream)
   if (M <= 8) {
     if (mode == OUT_BF16) Q3_GEMM_CASE(1, OUT_BF16);
     if (mode == OUT_F32) Q3_GEMM_CASE(1, OUT_F32);

@@ -66,7 +66,7 @@ template <bool HI> struct Blocks { static constexpr int value = 5; };
 template <int MODE, bool HI>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_stream_kernel(const bf16* __restrict__ x, int ldx, const bf16* __restrict__ W, int ldw, void* __restrict__ out,
-                   int ldo, int M, int N, int K, int up_offset, Plan plan, int* __restrict__ error_word) {
+                   int ldo, int M, int N, int K, int up_offset, int act, Plan plan, int* __restrict__ error_word) {
   constexpr int ROWS = 8;
   constexpr int XB = Blocks<HI>::value;
   constexpr int FPP = MODE == OUT_SWIGLU ? 4 : 8;  // output features per panel
@@ -164,7 +164,7 @@ gemm_stream_kernel(const bf16* __restrict__ x, int ldx, const bf16* __restrict__
       const int feature = panel * FPP + 2 * t + (e & 1);
       if (token < M && feature < N && (MODE != OUT_SWIGLU || t < 2)) {
         float r = v;
-        if (MODE == OUT_SWIGLU) r = (r / (1.f + expf(-r))) * up;
+        if (MODE == OUT_SWIGLU) r = gated_unit(r, up, act);
         if (MODE == OUT_PARTIAL)
           reinterpret_cast<float*>(out)[((long)part * M + token) * ldo + feature] = r;
         else if (MODE == OUT_F32)
@@ -234,7 +234,7 @@ bool make_plan(bool finished, int N, int K, int features_per_panel, int max_rang
 
 template <int MODE, bool HI>
 int launch(const bf16* x, int ldx, const bf16* W, int ldw, void* out, int ldo, int M, int N, int K, int up_offset,
-           int sm_count, int only_large, int planes, int* error_word, cudaStream_t stream) {
+           int act, int sm_count, int only_large, int planes, int* error_word, cudaStream_t stream) {
   const void* kernel = (const void*)gemm_stream_kernel<MODE, HI>;
   static bool configured_on[Q3_MAX_DEVICES];
   bool& configured = configured_on[q3_current_device()];
@@ -252,7 +252,7 @@ int launch(const bf16* x, int ldx, const bf16* W, int ldw, void* out, int ldo, i
   // per block) are faster on the kernel that streams through registers.
   if (MODE != OUT_PARTIAL && only_large && plan.panels < 8 * plan.blocks) return Q3_ERR_UNSUPPORTED;
   const size_t smem = (size_t)plan.stages * 8 * plan.pitch + RED_BYTES;
-  void* args[] = {&x, &ldx, &W, &ldw, &out, &ldo, &M, &N, &K, &up_offset, &plan, &error_word};
+  void* args[] = {&x, &ldx, &W, &ldw, &out, &ldo, &M, &N, &K, &up_offset, &act, &plan, &error_word};
   return launch_stream(kernel, plan.blocks, smem, stream, args) == cudaSuccess
              ? Q3_OK
              : Q3_ERR_LAUNCH;
@@ -273,14 +273,15 @@ int sm_count_of_current_device() {
 }  // namespace
 
 // mode 0: out bf16 [M, N]; 1: out fp32 [M, N]; 2: W is [2 * N, K] with gate rows first and up
-// rows from row `N`, out bf16 [M, N] = silu(x W_gate^T) * (x W_up^T).
+// rows from row `N`, out bf16 [M, N] = silu(x W_gate^T) * (x W_up^T); 3: the same with gelu (tanh form)
+// in place of silu.
 // M <= 16; K a multiple of 8 and at most 40960 (20480 when M > 8); leading dimensions in
 // elements (ldx, ldw multiples of 8); x and W 16-byte aligned; anything else is refused as
 // unsupported.  only_large != 0: also refuse the products for which q3_gemm_small_m is the
 // faster kernel on a B200.  `error_word` is set non-zero if a bounded wait expired.
 Q3_EXPORT int q3_gemm_stream(int mode, const void* x, int ldx, const void* W, int ldw, void* out, int ldo, int M,
                              int N, int K, int only_large, int* error_word, cudaStream_t stream) {
-  if (!x || !W || !out || !error_word || N < 1 || K < 1 || M < 0 || mode < 0 || mode > 2) return Q3_ERR_ARGUMENT;
+  if (!x || !W || !out || !error_word || N < 1 || K < 1 || M < 0 || mode < 0 || mode > 3) return Q3_ERR_ARGUMENT;
   if (M > 16 || K % 8 || ldx % 8 || ldw % 8 || ldx < K || ldw < K || ldo < N) return Q3_ERR_UNSUPPORTED;
   if (((uintptr_t)x | (uintptr_t)W) & 15) return Q3_ERR_UNSUPPORTED;
   if (M == 0) return Q3_OK;
@@ -288,10 +289,10 @@ Q3_EXPORT int q3_gemm_stream(int mode, const void* x, int ldx, const void* W, in
   if (!sms) return Q3_ERR_LAUNCH;
   const bf16* xp = (const bf16*)x;
   const bf16* wp = (const bf16*)W;
-  const int up = mode == OUT_SWIGLU ? N : 0;
+  const int act = mode == 3, up = mode >= OUT_SWIGLU ? N : 0;
 #define Q3_STREAM_CASE(MODE)                                                                                  \
-  return M > 8 ? launch<MODE, true>(xp, ldx, wp, ldw, out, ldo, M, N, K, up, sms, only_large, 0, error_word, stream)          \
-               : launch<MODE, false>(xp, ldx, wp, ldw, out, ldo, M, N, K, up, sms, only_large, 0, error_word, stream)
+  return M > 8 ? launch<MODE, true>(xp, ldx, wp, ldw, out, ldo, M, N, K, up, act, sms, only_large, 0, error_word, stream)          \
+               : launch<MODE, false>(xp, ldx, wp, ldw, out, ldo, M, N, K, up, act, sms, only_large, 0, error_word, stream)
   if (mode == OUT_BF16) Q3_STREAM_CASE(OUT_BF16);
   if (mode == OUT_F32) Q3_STREAM_CASE(OUT_F32);
   Q3_STREAM_CASE(OUT_SWIGLU);
@@ -321,6 +322,6 @@ Q3_EXPORT int q3_gemm_stream_partial(const void* x, int ldx, const void* W, int 
   if (!sms) return Q3_ERR_LAUNCH;
   const bf16* xp = (const bf16*)x;
   const bf16* wp = (const bf16*)W;
-  return M > 8 ? launch<OUT_PARTIAL, true>(xp, ldx, wp, ldw, out, N, M, N, K, 0, sms, 0, parts, error_word, stream)
-               : launch<OUT_PARTIAL, false>(xp, ldx, wp, ldw, out, N, M, N, K, 0, sms, 0, parts, error_word, stream);
+  return M > 8 ? launch<OUT_PARTIAL, true>(xp, ldx, wp, ldw, out, N, M, N, K, 0, 0, sms, 0, parts, error_word, stream)
+               : launch<OUT_PARTIAL, false>(xp, ldx, wp, ldw, out, N, M, N, K, 0, 0, sms, 0, parts, error_word, stream);
 }

@@ -72,7 +72,7 @@ template <int BN, int NB, int MODE>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ CUtensorMap tmap_w,
                     void* __restrict__ out, int ldo, int M, int N, int K, int up_row_offset,
-                    int* __restrict__ error_word) {
+                    int act, int* __restrict__ error_word) {
   constexpr int A_BYTES = BM * BK * 2;
   constexpr int B_BYTES = BN * BK * 2;
   constexpr int STAGE_BYTES = A_BYTES + NB * B_BYTES;
@@ -194,10 +194,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
             tmem_load32(lane_addr + BN + c0, up);
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
-            for (int e = 0; e < 32; ++e) {
-              const float gate = __uint_as_float(acc[e]);
-              v[e] = (gate / (1.f + expf(-gate))) * __uint_as_float(up[e]);
-            }
+            for (int e = 0; e < 32; ++e) v[e] = gated_unit(__uint_as_float(acc[e]), __uint_as_float(up[e]), act);
           } else {
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
@@ -260,7 +257,7 @@ template <int MODE>
 __global__ void __launch_bounds__(THREADS, 1)
 gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ CUtensorMap tmap_w,
                          void* __restrict__ out, int ldo, int M, int N, int K, int up_row_offset,
-                         int* __restrict__ error_word) {
+                         int act, int* __restrict__ error_word) {
   constexpr int A_BYTES = BM * BK * 2;       // this CTA's 128 token rows
   constexpr int B_BYTES = 128 * BK * 2;      // this CTA's 128 feature rows
   constexpr int STAGE_BYTES = A_BYTES + B_BYTES;
@@ -380,10 +377,7 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap tmap_a, const __gri
             tmem_load32(lane_addr + 128 + c0, up);
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
-            for (int e = 0; e < 32; ++e) {
-              const float gate = __uint_as_float(acc[e]);
-              v[e] = (gate / (1.f + expf(-gate))) * __uint_as_float(up[e]);
-            }
+            for (int e = 0; e < 32; ++e) v[e] = gated_unit(__uint_as_float(acc[e]), __uint_as_float(up[e]), act);
           } else {
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
@@ -574,7 +568,7 @@ int sm_count() {
 
 template <int BN, int NB, int MODE>
 int launch(const CUtensorMap& ta, const CUtensorMap& tw, void* out, int ldo, int M, int N, int K, int up_offset,
-           int* error_word, cudaStream_t stream) {
+           int act, int* error_word, cudaStream_t stream) {
   constexpr size_t smem = (size_t)STAGES * (BM * BK * 2 + NB * BN * BK * 2) + 1024;
   static bool configured_on[Q3_MAX_DEVICES];
   bool& configured = configured_on[q3_current_device()];
@@ -587,13 +581,13 @@ int launch(const CUtensorMap& ta, const CUtensorMap& tw, void* out, int ldo, int
   const int num_sms = sm_count();
   const int tiles = ((N + BN - 1) / BN) * ((M + BM - 1) / BM);
   const int grid = tiles < num_sms ? tiles : num_sms;  // one persistent block per SM
-  gemm_tcgen05_kernel<BN, NB, MODE><<<grid, THREADS, smem, stream>>>(ta, tw, out, ldo, M, N, K, up_offset, error_word);
+  gemm_tcgen05_kernel<BN, NB, MODE><<<grid, THREADS, smem, stream>>>(ta, tw, out, ldo, M, N, K, up_offset, act, error_word);
   return q3_launch_status();
 }
 
 template <int MODE>
 int launch_pair(const CUtensorMap& ta, const CUtensorMap& tw, void* out, int ldo, int M, int N, int K, int up_offset,
-                int* error_word, cudaStream_t stream) {
+                int act, int* error_word, cudaStream_t stream) {
   constexpr size_t smem = (size_t)PAIR_STAGES * (BM * BK * 2 + 128 * BK * 2) + 1024;
   static bool configured_on[Q3_MAX_DEVICES];
   bool& configured = configured_on[q3_current_device()];
@@ -630,7 +624,7 @@ int launch_pair(const CUtensorMap& ta, const CUtensorMap& tw, void* out, int ldo
   const int tiles = ((N + TILE_N - 1) / TILE_N) * ((M + 2 * BM - 1) / (2 * BM));
   cfg.gridDim = dim3(2 * (tiles < pairs ? tiles : pairs));
   const cudaError_t err = cudaLaunchKernelEx(&cfg, gemm_tcgen05_pair_kernel<MODE>, ta, tw, out, ldo, M, N, K,
-                                             up_offset, error_word);
+                                             up_offset, act, error_word);
   return err == cudaSuccess ? Q3_OK : Q3_ERR_LAUNCH;
 }
 
@@ -695,10 +689,12 @@ int launch_pair_wide(const CUtensorMap& ta, const CUtensorMap& tw, void* out, in
 // arguments and modes as q3_gemm_tcgen05.
 Q3_EXPORT int q3_gemm_tcgen05_pair(int mode, const void* x, int ldx, const void* W, int ldw, void* out, int ldo,
                                    int M, int N, int K, int* error_word, cudaStream_t stream) {
-  if (!x || !W || !out || N < 1 || K < 1 || M < 0 || mode < 0 || mode > 2) return Q3_ERR_ARGUMENT;
+  if (!x || !W || !out || N < 1 || K < 1 || M < 0 || mode < 0 || mode > 3) return Q3_ERR_ARGUMENT;
   if (ldx % 8 || ldw % 8 || ldx < K || ldw < K || ldo < N) return Q3_ERR_UNSUPPORTED;
   if (((uintptr_t)x | (uintptr_t)W) & 15) return Q3_ERR_UNSUPPORTED;
   if (M == 0) return Q3_OK;
+  const int act = mode == 3;  // gelu in place of silu
+  if (act) mode = OUT_SWIGLU;
   CUtensorMap ta, tw;
   const long w_rows = mode == OUT_SWIGLU ? 2L * N : N;
   if (mode != OUT_SWIGLU) {
@@ -715,13 +711,14 @@ Q3_EXPORT int q3_gemm_tcgen05_pair(int mode, const void* x, int ldx, const void*
     }
   }
   if (!q3_bf16_map(&ta, x, M, K, ldx, BM) || !q3_bf16_map(&tw, W, w_rows, K, ldw, 128)) return Q3_ERR_LAUNCH;
-  if (mode == OUT_SWIGLU) return launch_pair<OUT_SWIGLU>(ta, tw, out, ldo, M, N, K, N, error_word, stream);
-  if (mode == OUT_F32) return launch_pair<OUT_F32>(ta, tw, out, ldo, M, N, K, 0, error_word, stream);
-  return launch_pair<OUT_BF16>(ta, tw, out, ldo, M, N, K, 0, error_word, stream);
+  if (mode == OUT_SWIGLU) return launch_pair<OUT_SWIGLU>(ta, tw, out, ldo, M, N, K, N, act, error_word, stream);
+  if (mode == OUT_F32) return launch_pair<OUT_F32>(ta, tw, out, ldo, M, N, K, 0, 0, error_word, stream);
+  return launch_pair<OUT_BF16>(ta, tw, out, ldo, M, N, K, 0, 0, error_word, stream);
 }
 
 // mode 0: out bf16 [M, N]; 1: out fp32 [M, N]; 2: W is [2 * N, K] (gate rows, then up rows from
-// row N), out bf16 [M, N] = silu(x W_gate^T) * (x W_up^T).  x, W bf16 with 16-byte aligned bases
+// row N), out bf16 [M, N] = silu(x W_gate^T) * (x W_up^T); 3: the same with gelu (tanh form) in place of
+// silu.  x, W bf16 with 16-byte aligned bases
 // and row strides (elements) that are multiples of 8.  error_word: device int, set to 1 if a
 // wait inside the kernel expired (may be null).
 Q3_EXPORT int q3_gemm_tcgen05(int mode, const void* x, int ldx, const void* W, int ldw, void* out, int ldo, int M,
@@ -730,6 +727,8 @@ Q3_EXPORT int q3_gemm_tcgen05(int mode, const void* x, int ldx, const void* W, i
   if (ldx % 8 || ldw % 8 || ldx < K || ldw < K || ldo < N) return Q3_ERR_UNSUPPORTED;
   if (((uintptr_t)x | (uintptr_t)W) & 15) return Q3_ERR_UNSUPPORTED;
   if (M == 0) return Q3_OK;
+  const int act = mode == 3;
+  if (act) mode = OUT_SWIGLU;
   CUtensorMap ta, tw;
   int bn = 128;
   if (mode != OUT_SWIGLU) {
@@ -748,11 +747,11 @@ Q3_EXPORT int q3_gemm_tcgen05(int mode, const void* x, int ldx, const void* W, i
   }
   const long w_rows = mode == OUT_SWIGLU ? 2L * N : N;
   if (!q3_bf16_map(&ta, x, M, K, ldx, BM) || !q3_bf16_map(&tw, W, w_rows, K, ldw, bn)) return Q3_ERR_LAUNCH;
-  if (mode == OUT_SWIGLU) return launch<128, 2, OUT_SWIGLU>(ta, tw, out, ldo, M, N, K, N, error_word, stream);
+  if (mode == OUT_SWIGLU) return launch<128, 2, OUT_SWIGLU>(ta, tw, out, ldo, M, N, K, N, act, error_word, stream);
 #define Q3_TC_CASE(BN_)                                                                                   \
   if (bn == BN_)                                                                                          \
-    return mode == OUT_F32 ? launch<BN_, 1, OUT_F32>(ta, tw, out, ldo, M, N, K, 0, error_word, stream)    \
-                           : launch<BN_, 1, OUT_BF16>(ta, tw, out, ldo, M, N, K, 0, error_word, stream)
+    return mode == OUT_F32 ? launch<BN_, 1, OUT_F32>(ta, tw, out, ldo, M, N, K, 0, 0, error_word, stream)    \
+                           : launch<BN_, 1, OUT_BF16>(ta, tw, out, ldo, M, N, K, 0, 0, error_word, stream)
   if (mode == OUT_BF16 || mode == OUT_F32) {
     Q3_TC_CASE(256);
     Q3_TC_CASE(192);

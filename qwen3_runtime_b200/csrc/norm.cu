@@ -194,20 +194,20 @@ Q3_EXPORT int q3_fused_norm(int dtype, const void* pending, int pending_parts, l
   return Q3_ERR_ARGUMENT;
 }
 
-// ---- SwiGLU product: out[t, i] = silu(gu[t, i]) * gu[t, I + i]  (layers/ops.py:23-25) ----
+// ---- gated unit: out[t, i] = act(gu[t, i]) * gu[t, I + i], act silu (layers/ops.py:23-25) or gelu in its tanh form ----
 template <typename T>
-__global__ void silu_mul_kernel(const T* __restrict__ gu, T* __restrict__ out, long total, int I) {
+__global__ void glu_mul_kernel(const T* __restrict__ gu, T* __restrict__ out, long total, int I, int act) {
   const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= total) return;
   const long t = idx / I;
   const int i = (int)(idx - t * I);
   const float g = to_f32(gu[t * 2 * I + i]);
   const float u = to_f32(gu[t * 2 * I + I + i]);
-  out[idx] = from_f32<T>((g / (1.f + expf(-g))) * u);
+  out[idx] = from_f32<T>(gated_unit(g, u, act));
 }
 
 template <typename T>
-__global__ void silu_mul_vec_kernel(const T* __restrict__ gu, T* __restrict__ out, long chunks, int I) {
+__global__ void glu_mul_vec_kernel(const T* __restrict__ gu, T* __restrict__ out, long chunks, int I, int act) {
   const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= chunks) return;
   const int per_row = I / 8;
@@ -217,12 +217,13 @@ __global__ void silu_mul_vec_kernel(const T* __restrict__ gu, T* __restrict__ ou
   load8(gu + t * 2 * I + i, g);
   load8(gu + t * 2 * I + I + i, u);
 #pragma unroll
-  for (int e = 0; e < 8; ++e) g[e] = (g[e] / (1.f + expf(-g[e]))) * u[e];
+  for (int e = 0; e < 8; ++e) g[e] = gated_unit(g[e], u[e], act);
   store8(out + t * I + i, g);
 }
 
-Q3_EXPORT int q3_silu_mul(int dtype, const void* gu, void* out, int num_rows, int I, cudaStream_t stream) {
-  if (!gu || !out || I < 1) return Q3_ERR_ARGUMENT;
+// act 0: silu, 1: gelu (tanh form).
+Q3_EXPORT int q3_glu_mul(int dtype, const void* gu, void* out, int num_rows, int I, int act, cudaStream_t stream) {
+  if (!gu || !out || I < 1 || act < 0 || act > 1) return Q3_ERR_ARGUMENT;
   const long total = (long)num_rows * I;
   if (total == 0) return Q3_OK;
   const int threads = 256;
@@ -230,18 +231,18 @@ Q3_EXPORT int q3_silu_mul(int dtype, const void* gu, void* out, int num_rows, in
     const long chunks = total / 8;
     const unsigned vblocks = (unsigned)((chunks + threads - 1) / threads);
     if (dtype == Q3_DTYPE_F32)
-      silu_mul_vec_kernel<float><<<vblocks, threads, 0, stream>>>((const float*)gu, (float*)out, chunks, I);
+      glu_mul_vec_kernel<float><<<vblocks, threads, 0, stream>>>((const float*)gu, (float*)out, chunks, I, act);
     else if (dtype == Q3_DTYPE_BF16)
-      silu_mul_vec_kernel<bf16><<<vblocks, threads, 0, stream>>>((const bf16*)gu, (bf16*)out, chunks, I);
+      glu_mul_vec_kernel<bf16><<<vblocks, threads, 0, stream>>>((const bf16*)gu, (bf16*)out, chunks, I, act);
     else
       return Q3_ERR_ARGUMENT;
     return q3_launch_status();
   }
   const long blocks = (total + threads - 1) / threads;
   if (dtype == Q3_DTYPE_F32)
-    silu_mul_kernel<float><<<(unsigned)blocks, threads, 0, stream>>>((const float*)gu, (float*)out, total, I);
+    glu_mul_kernel<float><<<(unsigned)blocks, threads, 0, stream>>>((const float*)gu, (float*)out, total, I, act);
   else if (dtype == Q3_DTYPE_BF16)
-    silu_mul_kernel<bf16><<<(unsigned)blocks, threads, 0, stream>>>((const bf16*)gu, (bf16*)out, total, I);
+    glu_mul_kernel<bf16><<<(unsigned)blocks, threads, 0, stream>>>((const bf16*)gu, (bf16*)out, total, I, act);
   else
     return Q3_ERR_ARGUMENT;
   return q3_launch_status();

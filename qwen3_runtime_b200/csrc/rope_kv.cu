@@ -256,13 +256,16 @@ Q3_EXPORT int q3_rope_table(const float* inv_freq, float* cos_t, float* sin_t, i
 // square and multiplied by the one weight of D / maps elements.  `inv_freq` (fp32 [rot_half]): the first
 // 2 * rot_half elements of every part turn by angle = float(position) * inv_freq[i] (exact cosf/sinf, no
 // table, so no position is out of reach), pair i = (i, i + rot_half) with pairing 0 and (2i, 2i + 1) with
-// pairing 1; cos and sin are multiplied by `magnitude`.
+// pairing 1; cos and sin are multiplied by `magnitude`.  `q_scale` (fp32 [num_tokens], or null): a token's queries are
+// multiplied by its factor at the end.  `v_first` (rows v_first_stride apart with nv heads of Dv, or null): what is stored
+// as a token's value is (1 - v_share) * v + v_share * v_first (fp32, one rounding).
 template <typename T, int WARPS>
 __global__ void qk_norm_store_kernel(T* __restrict__ proj, long row_stride, int nq, int nkv, int nv, int D, int Dv,
                                      int k_start, int v_start, const float* __restrict__ q_w,
                                      const float* __restrict__ k_w, float eps, int maps,
                                      const float* __restrict__ inv_freq, int rot_half, int pairing, float magnitude,
-                                     const int* __restrict__ positions,
+                                     const float* __restrict__ q_scale, const T* __restrict__ v_first,
+                                     long v_first_stride, float v_share, const int* __restrict__ positions,
                                      const int* __restrict__ token_seq, const int* __restrict__ block_table,
                                      int max_pages, T* __restrict__ kpages, T* __restrict__ vpages, int ps,
                                      int num_tokens, int write_kv) {
@@ -286,16 +289,24 @@ __global__ void qk_norm_store_kernel(T* __restrict__ proj, long row_stride, int 
     if (page < 0) return;
     slot = ((long)page * (is_k ? nkv : nv) + kvh) * ps + (p % ps);
   }
-  if (hi >= nq + nkv) {  // value head: plain copy
-    const T* x = row + v_start + (long)(hi - nq - nkv) * Dv;
+  if (hi >= nq + nkv) {  // value head: a copy, or a blend with the first rows' head
+    const int vh = hi - nq - nkv;
+    const T* x = row + v_start + (long)vh * Dv;
     T* dst = vpages + slot * Dv;
+    if (v_first) {
+      const T* f = v_first + (long)t * v_first_stride + (long)vh * Dv;
+      for (int d = lane; d < Dv; d += 32)
+        dst[d] = from_f32<T>((1.f - v_share) * to_f32(x[d]) + v_share * to_f32(f[d]));
+      return;
+    }
     for (int d = lane; d < Dv; d += 32) dst[d] = x[d];
     return;
   }
   T* x = hi < nq ? row + (long)hi * D : row + k_start + (long)(hi - nq) * D;
   T* dst = hi < nq ? x : kpages + slot * D;
   const float* w = hi < nq ? q_w : k_w;
-  if (!w && !inv_freq) {
+  const float factor = hi < nq && q_scale ? q_scale[t] : 1.f;
+  if (!w && !inv_freq && factor == 1.f) {
     if (dst != x)
       for (int d = lane; d < D; d += 32) dst[d] = x[d];
     return;
@@ -325,19 +336,21 @@ __global__ void qk_norm_store_kernel(T* __restrict__ proj, long row_stride, int 
       const float yp = xs[d - dm + pd];
       y = first ? y * cs - yp * sn : y * cs + yp * sn;
     }
-    dst[d] = from_f32<T>(y);
+    dst[d] = from_f32<T>(y * factor);
   }
 }
 
 Q3_EXPORT int q3_qk_norm_store(int dtype, void* proj, long row_stride, int nq, int nkv, int nv, int D, int Dv,
                                int k_start, int v_start, const float* q_w, const float* k_w, float eps, int maps,
                                const float* inv_freq, int rot_half, int pairing, float magnitude,
+                               const float* q_scale, const void* v_first, long v_first_stride, float v_share,
                                const int* positions, const int* token_seq, const int* block_table, int max_pages,
                                void* kpages, void* vpages, int ps, int num_tokens, int write_kv,
                                cudaStream_t stream) {
   if (!proj || !positions || nq < 1 || nkv < 1 || nv < 1 || D < 1 || Dv < 1 || ps < 1) return Q3_ERR_ARGUMENT;
   if (maps < 1 || D % maps || pairing < 0 || pairing > 1) return Q3_ERR_ARGUMENT;
   if (inv_freq && (rot_half < 1 || 2 * rot_half > D / maps)) return Q3_ERR_ARGUMENT;
+  if (v_first && v_first_stride < (long)nv * Dv) return Q3_ERR_ARGUMENT;
   if (write_kv && (!token_seq || !block_table || !kpages || !vpages || max_pages < 1)) return Q3_ERR_ARGUMENT;
   if (num_tokens == 0) return Q3_OK;
   constexpr int WARPS = 4;
@@ -349,16 +362,38 @@ Q3_EXPORT int q3_qk_norm_store(int dtype, void* proj, long row_stride, int nq, i
   if (dtype == Q3_DTYPE_F32)
     e = launch_pdl(qk_norm_store_kernel<float, WARPS>, dim3(blocks), dim3(WARPS * 32), smem, stream, (float*)proj,
                    row_stride, nq, nkv, nv, D, Dv, k_start, v_start, q_w, k_w, eps, maps, inv_freq, rot_half, pairing,
-                   magnitude, positions, token_seq, block_table, max_pages, (float*)kpages, (float*)vpages, ps,
+                   magnitude, q_scale, (const float*)v_first, v_first_stride, v_share, positions, token_seq,
+                   block_table, max_pages, (float*)kpages, (float*)vpages, ps,
                    num_tokens, write_kv);
   else if (dtype == Q3_DTYPE_BF16)
     e = launch_pdl(qk_norm_store_kernel<bf16, WARPS>, dim3(blocks), dim3(WARPS * 32), smem, stream, (bf16*)proj,
                    row_stride, nq, nkv, nv, D, Dv, k_start, v_start, q_w, k_w, eps, maps, inv_freq, rot_half, pairing,
-                   magnitude, positions, token_seq, block_table, max_pages, (bf16*)kpages, (bf16*)vpages, ps,
+                   magnitude, q_scale, (const bf16*)v_first, v_first_stride, v_share, positions, token_seq,
+                   block_table, max_pages, (bf16*)kpages, (bf16*)vpages, ps,
                    num_tokens, write_kv);
   else
     return Q3_ERR_ARGUMENT;
   return e == cudaSuccess ? Q3_OK : Q3_ERR_LAUNCH;
+}
+
+// ---- factors for the queries of a step's tokens, worked out once for all layers with the same constants ----
+// factors[t] = 1 + coef * ln(floor((position + 1) / every) + 1)
+__global__ void query_temperature_kernel(const int* __restrict__ positions, float coef, int every,
+                                         float* __restrict__ factors, int num_tokens) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x * blockDim.x + threadIdx.x;
+  if (t < num_tokens) factors[t] = 1.f + coef * logf((float)((positions[t] + 1) / every + 1));
+}
+
+Q3_EXPORT int q3_query_temperature(const int* positions, float coef, int every, float* factors, int num_tokens,
+                                   cudaStream_t stream) {
+  if (!positions || !factors || every < 1) return Q3_ERR_ARGUMENT;
+  if (num_tokens == 0) return Q3_OK;
+  return launch_pdl(query_temperature_kernel, dim3((unsigned)((num_tokens + 127) / 128)), dim3(128), 0, stream, positions,
+                    coef, every, factors, num_tokens) == cudaSuccess
+             ? Q3_OK
+             : Q3_ERR_LAUNCH;
 }
 
 // ---- rotations of a step's tokens, worked out once for all layers that turn by the same frequencies ----

@@ -6,3 +6,4 @@ from . import puladra  # noqa: F401
 from . import medilix  # noqa: F401
 from . import tabisun  # noqa: F401
 from . import pevazen  # noqa: F401
+from . import timopel  # noqa: F401

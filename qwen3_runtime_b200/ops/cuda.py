@@ -52,7 +52,7 @@ _SIGNATURES = {
     "norm": {
         "q3_fused_norm": [c_int, c_void_p, c_int, c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                           c_void_p, c_int, c_int, c_float, c_int, c_int, c_void_p],
-        "q3_silu_mul": [c_int, c_void_p, c_void_p, c_int, c_int, c_void_p],
+        "q3_glu_mul": [c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
         "q3_add_bias": [c_int, c_void_p, c_long, c_void_p, c_int, c_int, c_void_p],
         "q3_logit_scale_cap": [c_void_p, c_long, c_float, c_float, c_void_p],
         "q3_fused_post_norm": [c_int, c_void_p, c_int, c_long, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -94,7 +94,7 @@ _SIGNATURES = {
     },
     "experts": {
         "q3_route_top": [c_int, c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
-                         c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+                         c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
         "q3_group_slots": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
         "q3_expert_gate_up_tc": [c_void_p, c_long, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                  c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float, c_float, c_float, c_void_p],
@@ -117,8 +117,10 @@ _SIGNATURES = {
                                   c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
         "q3_rope_table": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p],
         "q3_qk_norm_store": [c_int, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
-                             c_void_p, c_float, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p, c_void_p,
-                             c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+                             c_void_p, c_float, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p, c_long,
+                             c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int,
+                             c_void_p],
+        "q3_query_temperature": [c_void_p, c_float, c_int, c_void_p, c_int, c_void_p],
         "q3_turn_table": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p],
         "q3_turn_store": [c_int, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
                           c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
@@ -146,7 +148,7 @@ _SIGNATURES = {
     "attention_generic": {
         "q3_paged_attention_generic": [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                        c_void_p, c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                                       c_int, c_int, c_int, c_float, c_void_p, c_long, c_int, c_float, c_void_p,
+                                       c_int, c_int, c_void_p, c_void_p, c_long, c_int, c_float, c_void_p,
                                        c_int, c_int, c_void_p],
         "q3_paged_attention_diff": [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                     c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
@@ -182,7 +184,7 @@ _SIGNATURES = {
                                       c_float, c_int, c_int, c_void_p, c_void_p, c_void_p],
         "q3_paged_attention_decode_sink": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                            c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                           c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p,
+                                           c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                            c_int, c_float, c_void_p],
         "q3_paged_attention_decode_fused": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                             c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
@@ -192,7 +194,8 @@ _SIGNATURES = {
                                                  c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                                                  c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_float,
                                                  c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int,
-                                                 c_int, c_float, c_void_p, c_int, c_float, c_int, c_void_p],
+                                                 c_void_p, c_void_p, c_int, c_float, c_int, c_void_p, c_void_p, c_int,
+                                                 c_float, c_void_p],
     },
     "attention_prefill": {
         "q3_paged_attention_prefill": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
@@ -200,20 +203,20 @@ _SIGNATURES = {
                                        c_void_p],
         "q3_paged_attention_prefill_sink": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                             c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int,
-                                            c_int, c_int, c_float, c_void_p, c_int, c_float, c_void_p],
+                                            c_int, c_void_p, c_void_p, c_int, c_float, c_void_p],
     },
     "attention_prefill_tc": {
         "q3_paged_attention_prefill_tc": [c_void_p, c_int, c_int, c_void_p, c_void_p, ctypes.c_long, c_void_p, c_int,
                                           c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                                          c_float, c_int, c_int, c_void_p, c_void_p, c_void_p],
+                                          c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
     },
     "attention_chunk": {
         "q3_chunk_attention_prefill": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                        c_void_p, c_long, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int,
-                                       c_int, c_void_p, c_int, c_int, c_void_p],
+                                       c_int, c_void_p, c_int, c_int, c_void_p, c_void_p],
         "q3_chunk_attention_decode": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                                       c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                      c_int, c_float, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
+                                      c_int, c_float, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p],
     },
     "gemm_f32": {
         "q3_gemm_f32": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
@@ -600,12 +603,16 @@ class CudaOps:
                    float(cap))
         return logits
 
-    def silu_mul(self, gate_up, out):
+    # the unit of a gated feed-forward: activation(gate) * up ("gelu": its tanh form)
+    GLU_ACTIVATIONS = {"silu": 0, "gelu": 1}
+
+    def glu_mul(self, gate_up, out, activation="silu"):
+        """``out = activation(gate) * up``; rows of ``gate_up`` are ``[gate | up]`` (csrc/norm.cu)."""
         I = out.shape[-1]
         if self.timing is not None:
             self._costs(3 * out.shape[0] * I * out.element_size())
-        self._call("norm", "q3_silu_mul", "silu_mul",
-                   _dtype_code(out.dtype), _ptr(gate_up), _ptr(out), out.shape[0], I)
+        self._call("norm", "q3_glu_mul", "glu_mul", _dtype_code(out.dtype), _ptr(gate_up), _ptr(out), out.shape[0], I,
+                   self.GLU_ACTIVATIONS[activation])
         return out
 
     def sigmoid_mul(self, x, gate):
@@ -999,7 +1006,7 @@ class CudaOps:
         return out
 
     # ---- routed experts (csrc/experts.cu) --------------------------------------------------------
-    def route_top(self, h, router, top, renormalize=False, score="sigmoid", correction=None, groups=None):
+    def route_top(self, h, router, top, renormalize=False, score="sigmoid", correction=None, groups=None, scale=1.0):
         """``(chosen int32 [T, top], weights float32 [T, top])``: the float32 router product, the
         ``top`` largest per token in descending order (chosen on the logits, which order the experts as
         their sigmoids do without the ties of a saturated sigmoid; lowest index on an exact tie).
@@ -1007,7 +1014,8 @@ class CudaOps:
         their sum); ``"softmax_chosen"``: the softmax over the chosen logits only; ``"softmax_all"``: s is
         the softmax over all outputs, the choice is made on ``s + correction`` (float32 ``[E]`` or None) among
         the outputs of the ``groups[1]`` best of ``groups[0]`` equal groups of neighbours (a group's score: its
-        largest choice score), and the weights are the chosen s (``renormalize``: over their sum + 1e-20)."""
+        largest choice score), and the weights are the chosen s (``renormalize``: over their sum + 1e-20).
+        ``scale``: the weights are multiplied by it at the end."""
         if score not in ("sigmoid", "softmax_chosen", "softmax_all"):
             raise KernelError(f"route_top: unknown score {score!r}")
         mode = 3 if score == "softmax_all" else (2 if score == "softmax_chosen" else int(bool(renormalize)))
@@ -1031,7 +1039,7 @@ class CudaOps:
         self.launches += 1  # two kernels: the logits, then the choice
         self._call("experts", "q3_route_top", "route_top", _dtype_code(h.dtype), _ptr(h), h.stride(0), _ptr(router),
                    T, E, W, top, mode, _ptr(logits), _ptr(chosen), _ptr(weights), _ptr(correction), count, keep,
-                   int(bool(renormalize)))
+                   int(bool(renormalize)), float(scale))
         return chosen, weights
 
     def routed_experts(self, h, chosen, weights, gate_up, down, *, limit=0.0, alpha=1.0, up_offset=0.0,
@@ -1150,7 +1158,8 @@ class CudaOps:
 
     def qk_norm_store(self, proj, *, num_heads, num_kv_heads, head_dim, value_dim, k_start, v_start, q_weight,
                       k_weight, eps, positions, token_seq, block_table, k_pages, v_pages, page_size, write_kv,
-                      maps=1, num_value_heads=None, inv_freq=None, pairing="half", magnitude=1.0):
+                      maps=1, num_value_heads=None, inv_freq=None, pairing="half", magnitude=1.0, q_scale=None,
+                      first_values=None, value_share=0.0):
         """Per-head q/k RMSNorm (weights float32 shared by the heads, or None: as they are), an optional
         rotation, and the write of k and v into their pages (csrc/rope_kv.cu).  A row of ``proj`` holds the
         query heads from column 0, the key heads from ``k_start`` and the value heads (``value_dim`` each) from
@@ -1158,7 +1167,10 @@ class CudaOps:
         ``maps``: a head is that many consecutive parts of ``head_dim / maps`` elements, each normalised by
         itself with the one weight of that size.  ``num_value_heads``: the values' head count when it is not the
         keys'.  ``inv_freq`` (float32 ``[pairs]``): the first ``2 * pairs`` elements of every part turn by
-        ``position * inv_freq[i]``, pairs as ``pairing`` says, cos and sin times ``magnitude``; no table."""
+        ``position * inv_freq[i]``, pairs as ``pairing`` says, cos and sin times ``magnitude``; no table.
+        ``q_scale`` (float32 ``[T]``, :meth:`query_temperature`): a token's queries are multiplied by its factor at the
+        end.  ``first_values`` ``[T, value heads * value_dim]`` (a view of wider rows will do): what is stored as a value is
+        ``(1 - value_share) * v + value_share * first_values``."""
         T = proj.shape[0]
         if proj.stride(1) != 1:
             raise KernelError("qk_norm_store: unit-stride rows")
@@ -1172,14 +1184,42 @@ class CudaOps:
         pairs = inv_freq.numel() if inv_freq is not None else 0
         if inv_freq is not None and (inv_freq.dtype != torch.float32 or 2 * pairs > head_dim // maps):
             raise KernelError("qk_norm_store: float32 inverse frequencies, at most half a map's size of them")
+        self._check_query_scale(q_scale, T)
+        self._check_first_values(first_values, T, nv * value_dim, proj.dtype)
         max_pages = block_table.shape[1] if block_table is not None else 0
         if self.timing is not None:
             self._costs(2 * T * ((num_heads + num_kv_heads) * head_dim + num_kv_heads * value_dim) * proj.element_size())
         self._call("rope_kv", "q3_qk_norm_store", "qk_norm_store", _dtype_code(proj.dtype), _ptr(proj), proj.stride(0),
                    num_heads, num_kv_heads, nv, head_dim, value_dim, int(k_start), int(v_start), _ptr(q_weight),
                    _ptr(k_weight), float(eps), maps, _ptr(inv_freq), pairs, self.PAIRINGS[pairing], float(magnitude),
-                   _ptr(positions), _ptr(token_seq), _ptr(block_table), max_pages,
+                   _ptr(q_scale), _ptr(first_values), first_values.stride(0) if first_values is not None else 0,
+                   float(value_share), _ptr(positions), _ptr(token_seq), _ptr(block_table), max_pages,
                    _ptr(k_pages), _ptr(v_pages), page_size, T, int(bool(write_kv)))
+
+    @staticmethod
+    def _check_query_scale(q_scale, T):
+        if q_scale is not None and (q_scale.dtype != torch.float32 or q_scale.numel() != T or not q_scale.is_contiguous()):
+            raise KernelError("query factors are a dense float32 vector, one number per token")
+
+    @staticmethod
+    def _check_first_values(first, T, width, dtype):
+        if first is not None and (first.dtype != dtype or first.shape != (T, width) or first.stride(1) != 1):
+            raise KernelError("first values are [tokens, value heads * value size] of the activations' type")
+
+    @staticmethod
+    def _check_sink(sink, heads):
+        if sink is not None and (sink.dtype != torch.float32 or sink.numel() != heads or not sink.is_contiguous()):
+            raise KernelError("sinks are a dense float32 vector, one score per head")
+
+    def query_temperature(self, positions, coef, every):
+        """float32 ``[T]``: ``1 + coef * ln(floor((position + 1) / every) + 1)`` for every token of the step."""
+        T = positions.shape[0]
+        out = torch.empty(T, dtype=torch.float32, device=positions.device)
+        if self.timing is not None:
+            self._costs(T * 8)
+        self._call("rope_kv", "q3_query_temperature", "query_temperature", _ptr(positions), float(coef), int(every),
+                   _ptr(out), T)
+        return out
 
     def turn_table(self, positions, inv_freq):
         """float32 ``[T, 2, n]``: cos and sin of ``position * inv_freq`` for every token of the step."""
@@ -1230,15 +1270,16 @@ class CudaOps:
         softcap)`` after the scale.  ``value_dim``:
         values have a size of their own (``v_pages`` ``[pages, kv heads, page, value_dim]``); ``out`` may
         then be a view of wider rows, head h at column ``h * value_dim``.  ``keep_first``: with a window, the
-        sequence's first tokens stay visible as well.  ``sink``: a score without a value that is added to the
-        softmax's denominator.  ``gate`` ``[T, heads * value_dim]`` (a view of wider rows will do): the result
+        sequence's first tokens stay visible as well.  ``sink`` (float32 ``[heads]``): per head a score without a value
+        that is added to the softmax's denominator.  ``gate`` ``[T, heads * value_dim]`` (a view of wider rows will do): the result
         is multiplied by its sigmoid."""
         T = out.shape[0]
         if head_dim > 256:
             raise KernelError(f"paged_attention: head_dim={head_dim} is not supported (sizes up to 256 are)")
         Dv = int(value_dim or head_dim)
         keep_first = int(keep_first or 0) if window else 0
-        plain = not keep_first and sink is None and gate is None  # what the tcgen05 kernel takes
+        self._check_sink(sink, num_heads)
+        plain = not keep_first and gate is None  # what the tcgen05 kernel takes
         dense = out.stride(0) == num_heads * Dv and Dv == head_dim
         extras = dict(keep_first=keep_first, sink=sink, gate=gate)
         chunk, softcap = int(chunk or 0), float(softcap or 0.0)
@@ -1279,7 +1320,7 @@ class CudaOps:
                     _ptr(q), q_stride, q.shape[0], _ptr(k_pages), _ptr(v_pages),
                     k_pages.shape[0] * num_kv_heads * page_size, _ptr(block_table), block_table.shape[1],
                     _ptr(step.kv_lens), _ptr(step.cu_seqlens), _ptr(out), step.num_seqs, pairs, num_heads,
-                    num_kv_heads, head_dim, page_size, float(scale), 1, 0, None,
+                    num_kv_heads, head_dim, page_size, float(scale), 1, 0, None, _ptr(sink),
                     _ptr(self._error_word(out.device)), self._stream())
                 if self.timing is not None:
                     self._costs(*self._attention_cost(step, num_heads, num_kv_heads, head_dim, out, prompts=True))
@@ -1298,7 +1339,7 @@ class CudaOps:
                            _ptr(q), q_stride, _ptr(k_pages), _ptr(v_pages), _ptr(block_table),
                            block_table.shape[1], _ptr(step.kv_lens), _ptr(step.cu_seqlens), _ptr(out),
                            step.num_seqs, work, num_heads, num_kv_heads, head_dim, page_size, float(scale),
-                           int(window or 0), 1, keep_first, int(sink is not None), float(sink or 0.0), _ptr(gate),
+                           int(window or 0), 1, keep_first, _ptr(sink), _ptr(gate),
                            gate.stride(0) if gate is not None else 0, softcap)
             if step.num_single:
                 singles = [kv for kv, n in zip(step.host_kv_lens, qlens) if n == 1]
@@ -1315,22 +1356,22 @@ class CudaOps:
                 and head_dim % 8 == 0 and Dv % 8 == 0 and num_heads // num_kv_heads <= 16 and q_stride % 8 == 0
                 and out.stride(0) % 2 == 0 and q.data_ptr() % 16 == 0 and out.data_ptr() % 4 == 0):
             return self._chunk_attention(q, q_stride, num_heads, num_kv_heads, head_dim, Dv, k_pages, v_pages, block_table,
-                                         out, page_size, scale, chunk, step, value_turns, pairing)
+                                         out, page_size, scale, chunk, step, value_turns, pairing, sink)
         if self.timing is not None and step is not None:
             self._costs(*self._attention_cost(step, num_heads, num_kv_heads, head_dim, out))
         self._call("attention_generic", "q3_paged_attention_generic", "paged_attention",
                    _dtype_code(out.dtype), _ptr(q), q_stride, _ptr(k_pages), _ptr(v_pages), _ptr(block_table),
                   block_table.shape[1], _ptr(token_seq), _ptr(positions), _ptr(out), out.stride(0), T, num_heads,
                   num_kv_heads, head_dim, Dv, page_size, float(scale), int(window or 0), int(keep_first or 0),
-                  int(sink is not None), float(sink or 0.0), _ptr(gate), gate.stride(0) if gate is not None else 0,
+                  _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0,
                   chunk, softcap, _ptr(value_turns), value_turns.shape[2] if value_turns is not None else 0,
                   self.PAIRINGS[pairing])
         return out
 
     def _chunk_attention(self, q, q_stride, H, G, D, Dv, k_pages, v_pages, block_table, out, page_size, scale, chunk, step,
-                         turns, pairing):
+                         turns, pairing, sink=None):
         """:meth:`paged_attention` in bfloat16 with keys and values of sizes of their own, under a chunked mask
-        (``chunk`` 0: none), values possibly turned: prompt portions on the tensor cores (tcgen05 where heads of 128 and
+        (``chunk`` 0: none), values possibly turned, sinks or none: prompt portions on the tensor cores (tcgen05 where heads of 128 and
         the page size allow it, csrc/attention_prefill_tc.cu, else csrc/attention_chunk.cu), one-token sequences in
         slices of their visible keys (csrc/attention_chunk.cu)."""
         group = H // G
@@ -1352,7 +1393,7 @@ class CudaOps:
                 launch = lambda: self._get("attention_prefill_tc", "q3_paged_attention_prefill_tc")(  # noqa: E731
                     _ptr(q), q_stride, q.shape[0], _ptr(k_pages), _ptr(v_pages), k_pages.shape[0] * G * page_size,
                     _ptr(block_table), block_table.shape[1], _ptr(step.kv_lens), _ptr(step.cu_seqlens), _ptr(out),
-                    step.num_seqs, work, H, G, D, page_size, float(scale), skip, chunk, _ptr(turns),
+                    step.num_seqs, work, H, G, D, page_size, float(scale), skip, chunk, _ptr(turns), _ptr(sink),
                     _ptr(self._error_word(out.device)), self._stream())
                 if cost:
                     cost(True)
@@ -1370,7 +1411,7 @@ class CudaOps:
                            _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1], _ptr(step.kv_lens),
                            _ptr(step.cu_seqlens), _ptr(out), out.stride(0), step.num_seqs,
                            sum(-(-n * group // 128) for n in served), H, G, D, Dv, page_size, float(scale), chunk, skip,
-                           _ptr(turns), pairs, self.PAIRINGS[pairing])
+                           _ptr(turns), pairs, self.PAIRINGS[pairing], _ptr(sink))
         if singles:
             # the slice count comes from an upper bound of the lengths (in a captured step: the block-table width it
             # was captured for), never from the lengths of the moment
@@ -1394,7 +1435,7 @@ class CudaOps:
                        _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1], _ptr(step.kv_lens),
                        _ptr(step.cu_seqlens), None if step.decode_only else _ptr(step.single_seqs), _ptr(out),
                        out.stride(0), _ptr(mid_o), _ptr(mid_lse), _ptr(tickets), singles, H, G, D, Dv, page_size,
-                       float(scale), chunk, splits, _ptr(turns), pairs, self.PAIRINGS[pairing])
+                       float(scale), chunk, splits, _ptr(turns), pairs, self.PAIRINGS[pairing], _ptr(sink))
         return out
 
     @staticmethod
@@ -1571,7 +1612,8 @@ class CudaOps:
                                max_kv_len, seq_list=None, num_splits=None, new_token=None, step=None,
                                merge_kernel=False, longest=None, keep_first=0, sink=None, gate=None, softcap=None):
         """Split-KV attention for sequences that bring one token each (csrc/attention_decode.cu).
-        ``new_token`` (q_weight, k_weight, eps, cos, sin, optionally pairing and values_are_keys): ``q`` is
+        ``new_token`` (q_weight, k_weight, eps, cos, sin, optionally pairing, values_are_keys, q_scale, first_values and
+        value_share, the last three as in :meth:`qk_norm_store`): ``q`` is
         the raw q/k/v projection (q/k only with values_are_keys: a key head as projected is its value) and the
         kernel also does the work of :meth:`qk_norm_rope_store` for the newest position of each sequence,
         ``kv_lens - 1``.  The slices of a sequence and kv head are merged
@@ -1583,6 +1625,7 @@ class CudaOps:
         ``keep_first``, ``sink``, ``gate``, ``softcap``: as in :meth:`paged_attention`."""
         if out.dtype != torch.bfloat16 or head_dim not in (64, 128, 256) or num_heads // num_kv_heads > 16:
             raise KernelError("paged_attention_decode: bfloat16, head_dim 64/128/256 and groups of at most 16 only")
+        self._check_sink(sink, num_heads)
         keep_first = int(keep_first or 0) if window else 0
         if window:
             max_kv_len = min(max_kv_len, int(window) + keep_first + 63)
@@ -1603,6 +1646,9 @@ class CudaOps:
             self._costs(*self._attention_cost(step, num_heads, num_kv_heads, head_dim, out, prompts=False))
         if new_token is not None:
             cos, sin = new_token["cos"], new_token["sin"]
+            q_scale, first = new_token.get("q_scale"), new_token.get("first_values")
+            self._check_query_scale(q_scale, out.shape[0])
+            self._check_first_values(first, out.shape[0], num_kv_heads * head_dim, out.dtype)
             self._call("attention_decode", "q3_paged_attention_decode_fused_sink", "paged_attention_decode_fused",
                        _ptr(q), q_stride, _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1],
                        _ptr(kv_lens), _ptr(cu_seqlens), _ptr(seq_list), _ptr(out), _ptr(mid_o), _ptr(mid_lse),
@@ -1610,15 +1656,15 @@ class CudaOps:
                        splits, _ptr(new_token["q_weight"]), _ptr(new_token["k_weight"]), float(new_token["eps"]),
                        _ptr(cos), _ptr(sin), cos.shape[0] if cos is not None else 0,
                        self.PAIRINGS[new_token.get("pairing", "half")], err, _ptr(tickets), _ptr(longest),
-                       keep_first, int(sink is not None), float(sink or 0.0), _ptr(gate),
-                       gate.stride(0) if gate is not None else 0, float(softcap or 0.0),
-                       int(bool(new_token.get("values_are_keys"))))
+                       keep_first, _ptr(sink), _ptr(gate), gate.stride(0) if gate is not None else 0,
+                       float(softcap or 0.0), int(bool(new_token.get("values_are_keys"))), _ptr(q_scale), _ptr(first),
+                       first.stride(0) if first is not None else 0, float(new_token.get("value_share") or 0.0))
             return out
         self._call("attention_decode", "q3_paged_attention_decode_sink", "paged_attention_decode",
                    _ptr(q), q_stride, _ptr(k_pages), _ptr(v_pages), _ptr(block_table), block_table.shape[1],
                    _ptr(kv_lens), _ptr(cu_seqlens), _ptr(seq_list), _ptr(out), _ptr(mid_o), _ptr(mid_lse),
                    num_seqs, num_heads, num_kv_heads, head_dim, page_size, float(scale), int(window or 0), splits,
-                   _ptr(tickets), _ptr(longest), keep_first, int(sink is not None), float(sink or 0.0), _ptr(gate),
+                   _ptr(tickets), _ptr(longest), keep_first, _ptr(sink), _ptr(gate),
                    gate.stride(0) if gate is not None else 0, float(softcap or 0.0))
         return out
 
@@ -1735,13 +1781,13 @@ class CudaOps:
             self.raise_if_kernel_error()
 
     def linear_tcgen05(self, x, weight, out=None, out_dtype=None, mode=None, pair=None):
-        """``x @ weight^T`` on tcgen05 tensor cores (csrc/gemm_tcgen05.cu).  ``mode=2``: SwiGLU with
-        ``weight = [W_gate; W_up]``, ``out`` is ``[M, I]``.  ``pair``: the kernel that runs each
+        """``x @ weight^T`` on tcgen05 tensor cores (csrc/gemm_tcgen05.cu).  ``mode=2``: SwiGLU (3: with
+        gelu) with ``weight = [W_gate; W_up]``, ``out`` is ``[M, I]``.  ``pair``: the kernel that runs each
         256-token tile on two SMs (cta_group::2); default: when there are more than 128 tokens."""
         M, K = x.shape
         if not self._tcgen05_ok(x, weight):
             raise KernelError("gemm_tcgen05: bfloat16 operands with 16-byte aligned rows (K multiple of 8) only")
-        if mode == 2:
+        if mode in (2, 3):
             N = weight.shape[0] // 2
             odt = x.dtype
         else:
@@ -1816,23 +1862,25 @@ class CudaOps:
                 and x.stride(0) % 8 == 0 and weight.stride(0) % 8 == 0 and x.stride(1) == 1
                 and weight.stride(1) == 1 and x.data_ptr() % 16 == 0 and weight.data_ptr() % 16 == 0)
 
-    def gated_linear(self, x, gate_up_weight, out):
-        """``out = silu(x @ W_gate^T) * (x @ W_up^T)`` with ``gate_up_weight = [W_gate; W_up]``:
-        one kernel for a handful of tokens, else the product followed by the SwiGLU kernel."""
+    def gated_linear(self, x, gate_up_weight, out, activation="silu"):
+        """``out = act(x @ W_gate^T) * (x @ W_up^T)`` with ``gate_up_weight = [W_gate; W_up]``, act silu or gelu
+        (tanh form): one kernel for a handful of tokens and for prompt-sized batches, else the product followed by the
+        gated unit's kernel."""
         M, K = x.shape
         I = out.shape[1]
+        act = self.GLU_ACTIVATIONS[activation]
         if self.timing is not None:
             e = x.element_size()
             self._costs((2 * I * K + M * K + M * I) * e, 4.0 * M * I * K, f" {M}x{K}->2x{I} swiglu")
         if self._small_m_ok(x, gate_up_weight):
-            self._small_product(2, x, gate_up_weight, out, M, I, K)
+            self._small_product(2 + act, x, gate_up_weight, out, M, I, K)
             return out
         if self.large_gemm != "library" and self._tcgen05_ok(x, gate_up_weight):
             _pair, token_fill, share = self._tcgen05_plan(M, I)
             if self.large_gemm == "tcgen05" or (token_fill >= self.TCGEN05_MIN_TOKEN_FILL
                                                 and share >= self.TCGEN05_MIN_SHARE):
-                return self.linear_tcgen05(x, gate_up_weight, out=out, mode=2)
-        return self.silu_mul(self.linear(x, gate_up_weight), out)
+                return self.linear_tcgen05(x, gate_up_weight, out=out, mode=2 + act)
+        return self.glu_mul(self.linear(x, gate_up_weight), out, activation)
 
     # ---- sampling ---------------------------------------------------------------------
     def argmax(self, logits, want_logprob=False):

@@ -22,7 +22,7 @@ first product).
 ``correction`` per output (when ``correction`` is set), the weights are the chosen s themselves
 (``renormalize`` divides them by their sum + 1e-20).  ``groups = (count, keep)``: the router outputs form
 ``count`` equal groups of neighbours, a group's score is the largest choice score in it, and only outputs
-of the ``keep`` best groups can be chosen.  ``num_identity``: that many further router outputs (after the
+of the ``keep`` best groups can be chosen.  ``weight_scale``: a factor on all weights.  ``num_identity``: that many further router outputs (after the
 stored experts') stand for experts that return their input; they have no tensors.
 
 Tokens are grouped by expert on the device (no host round trip, so a step with experts can be
@@ -59,6 +59,7 @@ class RoutedExperts(Part):
             self.limit, self.alpha, self.up_offset = float("inf"), 1.0, 0.0
         self.score = spec.get("score", "sigmoid")
         self.renormalize = bool(spec.get("renormalize", False))
+        self.weight_scale = float(spec.get("weight_scale", 1.0))
         self.weight_on = spec.get("weight_on", "input")
         self.shared_size = int(spec["shared_size"]) if spec.get("shared_size") else 0
         self.shared_limit = float(spec.get("shared_limit") or self.limit)
@@ -136,9 +137,10 @@ class RoutedExperts(Part):
         ops = self.ops
         if self.score == "softmax_all":
             chosen, weights = ops.route_top(h, self.router, self.top, renormalize=self.renormalize, score=self.score,
-                                            correction=self.correction_vec, groups=self.groups)
+                                            correction=self.correction_vec, groups=self.groups, scale=self.weight_scale)
         else:
-            chosen, weights = ops.route_top(h, self.router, self.top, renormalize=self.renormalize, score=self.score)
+            chosen, weights = ops.route_top(h, self.router, self.top, renormalize=self.renormalize, score=self.score,
+                                            scale=self.weight_scale)
         shared = None
         if self.shared_size and not self.gated:
             up = ops.linear(h, self.shared_gate_up)

@@ -1,5 +1,6 @@
 """Dense gated feed-forward (SwiGLU): down(silu(gate x) * up x), no biases
-(qwen3_runtime/models/qwen3.py:130-138; layers/ops.py:23-25)."""
+(qwen3_runtime/models/qwen3.py:130-138; layers/ops.py:23-25).  ``activation="gelu"``: gelu in its tanh form in place
+of silu."""
 
 from __future__ import annotations
 
@@ -15,9 +16,9 @@ class GatedMLP(Part):
         super().__init__(spec, ctx)
         self.hidden_size = int(spec["hidden_size"])
         self.intermediate_size = int(spec["intermediate_size"])
-        activation = spec.get("activation", "silu")
-        if activation != "silu":
-            raise ValueError(f"gated_mlp has a silu kernel only, not {activation!r}")
+        self.activation = spec.get("activation", "silu")
+        if self.activation not in ("silu", "gelu"):
+            raise ValueError(f"gated_mlp has silu and gelu kernels, not {self.activation!r}")
         self.down_bias = bool(spec.get("down_bias", False))
         # the stored tensors' names (after the part's prefix), for checkpoints that call them otherwise
         names = dict(gate="gate_proj.weight", up="up_proj.weight", down="down_proj.weight",
@@ -51,7 +52,7 @@ class GatedMLP(Part):
 
     def forward(self, h: torch.Tensor, step: StepContext) -> torch.Tensor:
         mid = torch.empty((h.shape[0], self.intermediate_size), dtype=h.dtype, device=h.device)
-        self.ops.gated_linear(h, self.gate_up_weight, mid)
+        self.ops.gated_linear(h, self.gate_up_weight, mid, activation=self.activation)
         if self.down_bias_vec is not None:
             return self.ops.linear(mid, self.down_weight, bias=self.down_bias_vec)
         return self.ops.linear(mid, self.down_weight, partial_sums=self.partial_sums_ok)

@@ -1,6 +1,7 @@
 """RMSNorm: y = x * rsqrt(mean(x^2) + eps) * w, all in float32, one rounding at the end
 (qwen3_runtime/layers/ops.py:17-20; residual form :28-37).  ``weight_offset``: the stored weight
 is the deviation from this value, which is added to it when it is loaded (y = ... * (offset + w)).
+``weight_scale``: a factor on the norm's output, multiplied into the weight when it is loaded.
 ``groups`` > 1: a row is cut into that many equal consecutive parts and each is divided by its own root
 mean square (the weight still spans the whole row).
 ``scalar``: the stored weight is one number for all coordinates (a tensor without dimensions).
@@ -26,6 +27,7 @@ class RMSNorm(Part):
         # the stored tensor's name after the part's prefix ("" when the prefix is the whole name)
         self.weight_name = str(spec.get("weight_name", "weight"))
         self.weight_offset = float(spec.get("weight_offset", 0.0))
+        self.weight_scale = float(spec.get("weight_scale", 1.0))
         self.groups = int(spec.get("groups") or 1)
         self.scalar = bool(spec.get("scalar", False))
         if self.groups < 1 or self.size % self.groups:
@@ -43,6 +45,8 @@ class RMSNorm(Part):
             self.weight = self.weight.expand(self.size).contiguous()
         if self.weight_offset:
             self.weight = (self.weight.float() + self.weight_offset).contiguous()
+        if self.weight_scale != 1.0:
+            self.weight = (self.weight.float() * self.weight_scale).contiguous()
 
     def pending_scale(self) -> tuple:
         """This norm as something the next norm applies to what is pending (``ResidualStream.pending_norm``):

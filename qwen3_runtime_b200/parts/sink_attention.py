@@ -17,7 +17,11 @@ that many tokens counted from the sequence's first token); ``qkv_bias`` (biases 
 projections); ``own_kv=False`` (the layer has no key and value projections and reads the keys and values another
 layer has stored, under its own mask); ``value_turn`` (a rotary base: the value of position j is turned by j over
 all its dimensions before it is stored, pair m by ``j * base^(-2m / vdim)``, and a head's sum at position i is turned
-back by i).
+back by i); ``query_temperature`` ``(coef, every)`` (the normed and turned query of position p is multiplied by
+1 + coef * ln(floor((p + 1) / every) + 1)); ``value_mix`` (``"source"``: the layer's values as projected are kept for
+the later layers of the step; ``"blend"``: the layer's values become (1 - lambda) v + lambda v_source before they are
+stored, lambda being the stored number ``vmix``, which a source has too but does not use).  ``sink`` is one score for
+all heads (a number) or ``"learned"`` (one stored number per head, ``sink``).
 
 The part is a :class:`BranchMixer`: it runs alone or as a branch of the ``parallel`` mixer.
 """
@@ -43,7 +47,12 @@ class SinkWindowAttention(BranchMixer):
         self.scale = float(spec["scale"])
         self.window = spec.get("window") or None
         self.keep_first = int(spec.get("keep_first") or 0) if self.window else 0
-        self.sink = spec.get("sink")  # the sink's score (a number), or None
+        sink = spec.get("sink")  # one score for all heads (a number), "learned" (a stored score per head), or None
+        self.learned_sink = sink == "learned"
+        self.has_sink = sink is not None
+        self.sink = None  # float32 [heads]
+        if self.has_sink and not self.learned_sink:
+            self.sink = torch.full((self.num_heads,), float(sink), dtype=torch.float32, device=ctx.device)
         self.gate = spec.get("gate")  # "sigmoid" or None
         self.qk_norm_eps = spec.get("qk_norm_eps")
         if self.num_heads % self.num_kv_heads:
@@ -82,6 +91,16 @@ class SinkWindowAttention(BranchMixer):
         if not self.turned and (self.qkv_bias or not self.own_kv or self.value_position is not None):
             raise ValueError("sink_window_attention: biases, shared keys and turned values go without q/k norms and with "
                              "values of their own")
+        temperature = spec.get("query_temperature")
+        self.temperature = (float(temperature[0]), int(temperature[1])) if temperature else None
+        self.value_mix = spec.get("value_mix")
+        if self.value_mix not in (None, "source", "blend"):
+            raise ValueError(f"sink_window_attention: value_mix is 'source', 'blend' or absent, not {self.value_mix!r}")
+        if self.turned and (self.temperature or self.value_mix):
+            raise ValueError("sink_window_attention: a query temperature and mixed values go with q/k norms")
+        if self.values_are_keys and self.value_mix:
+            raise ValueError("sink_window_attention: values that are the keys are not mixed")
+        self.value_share = 0.0
         self.in_weight = self.o_weight = self.q_norm = self.k_norm = self.bias = None
         self._tables = None
         self.starts: list[int] = []
@@ -101,6 +120,10 @@ class SinkWindowAttention(BranchMixer):
         if self.qk_norm_eps is not None:
             specs["q.norm"] = ParamSpec((D,), "vector")
             specs["k.norm"] = ParamSpec((D,), "vector")
+        if self.value_mix:
+            specs["vmix"] = ParamSpec((), "vector")
+        if self.learned_sink:
+            specs["sink"] = ParamSpec((H,), "vector")
         return specs
 
     def load(self, tensors):
@@ -122,6 +145,10 @@ class SinkWindowAttention(BranchMixer):
         self.o_weight = tensors["o"].contiguous()
         self.q_norm = tensors.get("q.norm")
         self.k_norm = tensors.get("k.norm")
+        if self.learned_sink:
+            self.sink = tensors["sink"].contiguous()
+        if self.value_mix == "blend":
+            self.value_share = float(tensors["vmix"])
 
     def input_weight(self):
         return self.in_weight
@@ -138,8 +165,9 @@ class SinkWindowAttention(BranchMixer):
     def kernel_groups(self):
         groups = ["rope_kv", "attention_generic"]
         groups += ["gemm_f32"] if self.ctx.dtype == torch.float32 else ["gemm_small_m", "gemm_stream"]
-        if self.turned and self.ctx.dtype == torch.bfloat16 and not self.window and self.sink is None and not self.gate:
-            groups.append("attention_chunk")
+        if self.ctx.dtype == torch.bfloat16 and not self.window and not self.gate and not self.softcap:
+            if self.turned or not self._specialised() or self.dim == 256:
+                groups.append("attention_chunk")
             if self.dim == 128 and self.vdim == 128:
                 groups.append("attention_prefill_tc")
         if self._specialised():
@@ -203,6 +231,21 @@ class SinkWindowAttention(BranchMixer):
             step.extras[key] = self.ops.turn_table(step.positions, inv)
         return step.extras[key]
 
+    def _query_scale(self, step: StepContext):
+        """The factors of the step's queries, made by the first layer that asks for these constants."""
+        if self.temperature is None:
+            return None
+        key = ("query_temperature", *self.temperature)
+        if key not in step.extras:
+            step.extras[key] = self.ops.query_temperature(step.positions, *self.temperature)
+        return step.extras[key]
+
+    def _first_values(self, own, step: StepContext):
+        """The values this layer's are blended with (None: they stay as they are).  ``own``: its values as projected."""
+        if self.value_mix == "source":
+            step.extras["first_values"] = own
+        return step.extras["first_values"] if self.value_mix == "blend" else None
+
     def _turned_context(self, proj, step: StepContext, cache, ctx) -> None:
         ops = self.ops
         H, G, D, Dv = self.num_heads, self.num_kv_heads, self.dim, self.vdim
@@ -236,6 +279,10 @@ class SinkWindowAttention(BranchMixer):
         gate = proj[:, s[3]:s[3] + H * Dv] if self.gate else None
         fusable = getattr(ops, "decode_new_token_ok", None)
         rotary = self.position.style == "rotary"
+        blend = {}
+        if self.temperature or self.value_mix:
+            blend = dict(q_scale=self._query_scale(step), value_share=self.value_share,
+                         first_values=self._first_values(proj[:, s[2]:s[2] + G * Dv], step))
         tables = None
         if (fusable is not None and step.decode_only and cache.writes and self._specialised() and rotary
                 and (step.captured_width * cache.page_size or step.max_kv_len) <= self.FUSED_POSITIONS):
@@ -258,7 +305,7 @@ class SinkWindowAttention(BranchMixer):
                 new_token=dict(q_weight=self.q_norm, k_weight=self.k_norm,
                                eps=self.qk_norm_eps if self.qk_norm_eps is not None else 0.0, cos=cos, sin=sin,
                                pairing=getattr(self.position, "pairing", "half"),
-                               values_are_keys=self.values_are_keys),
+                               values_are_keys=self.values_are_keys, **blend),
                 num_splits=step.choices.get(self._slices_key()), longest=step.kv_longest, step=step,
                 keep_first=self.keep_first, sink=self.sink, gate=gate, softcap=self.softcap)
             return
@@ -268,7 +315,7 @@ class SinkWindowAttention(BranchMixer):
                           token_seq=step.token_seq, block_table=block_table, k_pages=cache.k_pages,
                           v_pages=cache.v_pages, page_size=cache.page_size, write_kv=cache.writes,
                           **(dict(inv_freq=self.position.inverse_frequencies(), pairing=self.position.pairing,
-                                  magnitude=getattr(self.position, "magnitude", 1.0)) if rotary else {}))
+                                  magnitude=getattr(self.position, "magnitude", 1.0)) if rotary else {}), **blend)
         ops.paged_attention(proj, proj.stride(0), num_heads=H, num_kv_heads=G, head_dim=D, k_pages=cache.k_pages,
                             v_pages=cache.v_pages, block_table=block_table, token_seq=step.token_seq,
                             positions=step.positions, out=ctx, page_size=cache.page_size, scale=self.scale,

@@ -276,7 +276,8 @@ class TorchOps:
 
     def qk_norm_store(self, proj, *, num_heads, num_kv_heads, head_dim, value_dim, k_start, v_start, q_weight, k_weight,
                       eps, positions, token_seq, block_table, k_pages, v_pages, page_size, write_kv, maps=1,
-                      num_value_heads=None, inv_freq=None, pairing="half", magnitude=1.0):
+                      num_value_heads=None, inv_freq=None, pairing="half", magnitude=1.0, q_scale=None, first_values=None,
+                      value_share=0.0):
         T = proj.shape[0]
         H, G, D, Dv = num_heads, num_kv_heads, head_dim, value_dim
         Gv = int(num_value_heads or G)
@@ -292,7 +293,12 @@ class TorchOps:
 
         raw_k = proj[:, k_start:k_start + G * D].reshape(T, G, D).float()
         raw_v = proj[:, v_start:v_start + Gv * Dv].reshape(T, Gv, Dv).clone()
+        if first_values is not None:
+            raw_v = ((1.0 - value_share) * raw_v.float()
+                     + value_share * first_values.reshape(T, Gv, Dv).float()).to(proj.dtype)
         q = unit(proj[:, : H * D].reshape(T, H, D).float(), q_weight)
+        if q_scale is not None:
+            q = q * q_scale[:, None, None]
         proj[:, : H * D] = q.reshape(T, H * D).to(proj.dtype)
         if not write_kv:
             return
@@ -304,6 +310,9 @@ class TorchOps:
                 continue
             k_pages[page, :, p % page_size, :] = k[t]
             v_pages[page, :, p % page_size, :] = raw_v[t]
+
+    def query_temperature(self, positions, coef, every):
+        return 1.0 + coef * torch.log(((positions.long() + 1) // every + 1).float())
 
     @staticmethod
     def _turn_pairs(x, pos, inv_freq, pairing, magnitude=1.0):
@@ -326,10 +335,11 @@ class TorchOps:
             out[..., pairs:2 * pairs] = v * c + u * s
         return out
 
-    def silu_mul(self, gate_up, out):
+    def glu_mul(self, gate_up, out, activation="silu"):
         I = out.shape[-1]
         g, u = gate_up[:, :I].float(), gate_up[:, I:].float()
-        out.copy_(((g / (1 + torch.exp(-g))) * u).to(out.dtype))
+        a = torch.nn.functional.gelu(g, approximate="tanh") if activation == "gelu" else g / (1 + torch.exp(-g))
+        out.copy_((a * u).to(out.dtype))
         return out
 
     def relu_squared(self, x, out):
@@ -508,7 +518,7 @@ class TorchOps:
             if softcap:
                 scores = softcap * torch.tanh(scores / softcap)
             if sink is not None:  # one more score that has no value
-                scores = torch.cat([scores, torch.full((num_heads, 1), float(sink), device=scores.device)], dim=-1)
+                scores = torch.cat([scores, sink.float().reshape(num_heads, 1)], dim=-1)
                 probs = torch.softmax(scores, dim=-1)[:, :-1]
             else:
                 probs = torch.softmax(scores, dim=-1)
@@ -608,7 +618,12 @@ class TorchOps:
         return out
 
     # ---- routed experts ----------------------------------------------------------------
-    def route_top(self, h, router, top, renormalize=False, score="sigmoid", correction=None, groups=None):
+    def route_top(self, h, router, top, renormalize=False, score="sigmoid", correction=None, groups=None, scale=1.0):
+        chosen, w = self._route(h, router, top, renormalize, score, correction, groups)
+        return chosen, w * scale
+
+    @staticmethod
+    def _route(h, router, top, renormalize, score, correction, groups):
         if score == "softmax_all":
             s_all = torch.softmax(h.float() @ router.float().t(), dim=-1)
             choice = s_all + correction.float() if correction is not None else s_all.clone()
@@ -690,8 +705,8 @@ class TorchOps:
             return out
         return res
 
-    def gated_linear(self, x, gate_up_weight, out):
-        return self.silu_mul(self.linear(x, gate_up_weight), out)
+    def gated_linear(self, x, gate_up_weight, out, activation="silu"):
+        return self.glu_mul(self.linear(x, gate_up_weight), out, activation)
 
     # ---- sampling ---------------------------------------------------------------------
     def argmax(self, logits, want_logprob=False):

@@ -397,7 +397,7 @@ def case_attention_edges(dtype, ops, device, *, window=12, keep=3, page_size=8, 
             ops.paged_attention(qd, qd.stride(0), num_heads=heads, num_kv_heads=kv_heads, head_dim=D, k_pages=k_pages,
                                 v_pages=v_pages, block_table=step.block_tables[0], token_seq=step.token_seq,
                                 positions=step.positions, out=wide[:, pad:pad + heads * Dv], page_size=page_size, scale=1.0,
-                                window=win, step=step, value_dim=Dv, keep_first=kp, sink=0.0,
+                                window=win, step=step, value_dim=Dv, keep_first=kp, sink=torch.zeros(heads, device=device),
                                 gate=g[lo:hi].to(device=device, dtype=dt),
                                 **({"decode_slices": decode_slices} if decode_slices and hi - lo == 1 else {}))
             out = wide[:, pad:pad + heads * Dv].float().cpu().reshape(hi - lo, heads, Dv)

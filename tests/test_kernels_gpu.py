@@ -72,13 +72,14 @@ def test_fused_norm_variants(ops, dtype, H, T):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("I,T", [(9728, 5), (111, 64), (160, 1)])
-def test_silu_mul(ops, dtype, I, T):
+def test_glu_mul(ops, dtype, I, T):
     gu = rand((T, 2 * I), dtype, 6, scale=3.0)
     a = torch.empty((T, I), dtype=dtype, device="cuda")
     b = torch.empty_like(a)
-    ops.silu_mul(gu, a)
-    REF.silu_mul(gu, b)
-    close(a, b, dtype, "silu_mul", bf16_tol=1e-2)
+    for activation in ("silu", "gelu"):
+        ops.glu_mul(gu, a, activation)
+        REF.glu_mul(gu, b, activation)
+        close(a, b, dtype, f"glu_mul {activation}", bf16_tol=1e-2)
 
 
 def test_rope_table_matches_host_formula(ops):
@@ -678,6 +679,8 @@ def test_gated_linear_small_m(ops, small_gemm, M, I, K):
     ops.gated_linear(x, w, out)
     g, u = x.float() @ w[:I].float().t(), x.float() @ w[I:].float().t()
     close(out, torch.nn.functional.silu(g) * u, torch.bfloat16, "fused SwiGLU", bf16_tol=1e-2)
+    ops.gated_linear(x, w, out, activation="gelu")
+    close(out, torch.nn.functional.gelu(g, approximate="tanh") * u, torch.bfloat16, "fused GeGLU", bf16_tol=1e-2)
     # more tokens than the fused kernel takes: product, then the SwiGLU kernel
     xb = rand((40, K), torch.bfloat16, 59)
     outb = torch.empty((40, I), dtype=torch.bfloat16, device="cuda")
@@ -785,7 +788,7 @@ def test_kernels_refuse_sizes_they_do_not_support(ops):
     with pytest.raises(KernelError):
         ops.linear(torch.zeros(2, 8).cuda(), torch.zeros(4, 9).cuda())
     with pytest.raises(KernelError, match="float32 and bfloat16"):
-        ops.silu_mul(torch.zeros(2, 8, dtype=torch.float16).cuda(), torch.zeros(2, 4, dtype=torch.float16).cuda())
+        ops.glu_mul(torch.zeros(2, 8, dtype=torch.float16).cuda(), torch.zeros(2, 4, dtype=torch.float16).cuda())
 
 
 def test_a_bounded_wait_that_runs_out_is_reported_and_the_context_stays_usable(ops):
