@@ -59,6 +59,11 @@ kinds and a roofline fraction per kind):
                    rule, attention with biases and with another layer's keys, one norm per layer, averages over
                    the depth) at two layer sizes beside the Puladra design at equal sizes, its closest relative
                    (windowed attention beside retention, gated linear attention);
+* ``timopel``      the Timopel design (attention with normed q and k, a query temperature in place of positions, a
+                   learned sink per head and values mixed with the first layer's; gelu feed-forward and routed clamped
+                   experts with a shared one; norms around every sublayer) at three layer sizes beside the Medilix
+                   design (full attention with a sink and a gate, routed experts, a dense layer) and the Logesun design
+                   (norms around every sublayer, the same experts) at equal sizes, its closest relatives;
 * ``decode``, ``latency``, ``batch8``, ``throughput``, ``prefill``, ``longctx``: the six closed
                    batches of the reference's own harness (bench/workloads.py:34-43) at Qwen3-4B
                    sizes, with its token budget rule (bench/workloads.py:52-64).
@@ -110,7 +115,8 @@ BASELINE_TOK_S = 693.26
 # (concurrency = requests, prompt tokens, output tokens) of the reference's closed batches
 CLOSED_CASES = {"decode": (1, 256, 512), "latency": (1, 512, 128), "batch8": (8, 256, 128),
                 "throughput": (16, 256, 128), "prefill": (1, 2048, 16), "longctx": (1, 8192, 64)}
-WORKLOADS = ("default", "decode512", "batch48", "32b", "logesun", "puladra", "medilix", "tabisun", "pevazen", *CLOSED_CASES)
+WORKLOADS = ("default", "decode512", "batch48", "32b", "logesun", "puladra", "medilix", "tabisun", "pevazen", "timopel",
+             *CLOSED_CASES)
 
 # Layer sizes for the Puladra design that resemble real models of its kinds of layer: gated linear
 # attention with keys of half and values of the full width, windowed attention with grouped key/value
@@ -169,6 +175,19 @@ PEVAZEN_SIZES = {
                   delta=dict(heads=16, kv_heads=8, dim=128, vdim=128, conv=4, rank=64), experts=16, top=4),
     "w4096": dict(width=4096, ff=12288, vocab=32000, layers=4, chunk=2048, att=dict(heads=32, kv_heads=8, dim=128, rot=64),
                   delta=dict(heads=32, kv_heads=16, dim=128, vdim=128, conv=4, rank=128), experts=16, top=4),
+}
+
+# Layer sizes for the Timopel design: grouped heads of 128 (in the third size values of 96), a query temperature in steps of
+# 1,024 tokens, values mixed in every layer, one dense gelu feed-forward and three routed layers with a shared expert.
+# Beside each run Medilix (four full-attention layers with a sink and a gate, the same router, experts and dense width, no
+# shared expert) and Logesun (attention through a latent, the same dense and routed feed-forwards).
+TIMOPEL_SIZES = {
+    "w2048": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, dense_ff=8192, experts=64, top=6, expert_ff=1408,
+                  shared_ff=2816, layers=4, vocab=32000, rot_dim=64, q_rank=768, kv_rank=512, window=None),
+    "w4096": dict(width=4096, heads=32, kv_heads=8, dim=128, vdim=128, dense_ff=12288, experts=32, top=4, expert_ff=2048,
+                  shared_ff=2048, layers=4, vocab=32000, rot_dim=64, q_rank=1536, kv_rank=512, window=None),
+    "w2048v96": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=96, dense_ff=8192, experts=64, top=6, expert_ff=1408,
+                     shared_ff=2816, layers=4, vocab=32000, rot_dim=64, q_rank=768, kv_rank=512, window=None),
 }
 
 # Layer sizes for the Logesun design (attention through a latent with a window and a sink, routed
@@ -751,7 +770,7 @@ def _logesun_twin_config(z: dict):
 
 def run_tabisun(args, pk) -> dict:
     return run_design_beside_dense(args, pk, "tabisun", "Tabisun", TABISUN_SIZES, _tabisun_config,
-                                   twin=("logesun", _logesun_twin_config, "the Logesun design"))
+                                   twins=(("logesun", _logesun_twin_config, "the Logesun design"),))
 
 
 def _pevazen_config(z: dict):
@@ -799,7 +818,7 @@ def _puladra_beside_pevazen_config(z: dict):
 
 def run_pevazen(args, pk) -> dict:
     return run_design_beside_dense(args, pk, "pevazen", "Pevazen", PEVAZEN_SIZES, _pevazen_config,
-                                   twin=("puladra", _puladra_beside_pevazen_config, "the Puladra design"))
+                                   twins=(("puladra", _puladra_beside_pevazen_config, "the Puladra design"),))
 
 
 def _puladra_twin_config(z: dict):
@@ -815,7 +834,45 @@ def _puladra_twin_config(z: dict):
 
 def run_medilix(args, pk) -> dict:
     return run_design_beside_dense(args, pk, "medilix", "Medilix", MEDILIX_SIZES, _medilix_config,
-                                   twin=("puladra", _puladra_twin_config, "the Puladra design"))
+                                   twins=(("puladra", _puladra_twin_config, "the Puladra design"),))
+
+
+def _timopel_config(z: dict):
+    from qwen3_runtime_b200.config import TimopelConfig
+    from qwen3_runtime_b200.config.logesun_config import ExpertConfig
+    from qwen3_runtime_b200.config.timopel_config import (DenseConfig, MixedValueAttentionConfig, MoeConfig,
+                                                          TemperatureConfig, TimopelLayerConfig)
+
+    att = MixedValueAttentionConfig(heads=z["heads"], kv_heads=z["kv_heads"], dim=z["dim"], vdim=z["vdim"],
+                                    scale=z["dim"] ** -0.5, q_temp=TemperatureConfig(coef=0.1, every=1024), v_mix=True)
+    moe = MoeConfig(experts=z["experts"], top=z["top"], scale=1.0, expert=ExpertConfig(z["expert_ff"], 7.0),
+                    shared=ExpertConfig(z["shared_ff"], 7.0))
+    layers = tuple(TimopelLayerConfig("attention", att, DenseConfig(z["dense_ff"]) if i == 0 else moe)
+                   for i in range(z["layers"]))
+    return TimopelConfig(vocab=z["vocab"], width=z["width"], norm_eps=1e-6, layers=layers, embed_scale=4.0,
+                         residual_mult=0.5)
+
+
+def _medilix_beside_timopel_config(z: dict):
+    """Medilix at the sizes of a Timopel entry: full-attention layers only (values of the keys' size), the same router,
+    experts and dense width."""
+    from qwen3_runtime_b200.config import MedilixConfig
+    from qwen3_runtime_b200.config.medilix_config import (DenseConfig, GatedAttentionConfig, MedilixLayerConfig,
+                                                          MoeConfig)
+
+    att = GatedAttentionConfig(heads=z["heads"], kv_heads=z["kv_heads"], dim=z["dim"], vdim=z["dim"],
+                               scale=z["dim"] ** -0.5, window=None, keep_first=0)
+    moe = MoeConfig(experts=z["experts"], identity=0, top=z["top"], ff=z["expert_ff"], groups=1, groups_keep=1)
+    layers = tuple(MedilixLayerConfig("attention", att, DenseConfig(z["dense_ff"], 7.0) if i == 0 else moe)
+                   for i in range(z["layers"]))
+    return MedilixConfig(vocab=z["vocab"], width=z["width"], norm_eps=1e-6, norm_groups=1, embed_scale=1.0, bigram=None,
+                         layers=layers)
+
+
+def run_timopel(args, pk) -> dict:
+    return run_design_beside_dense(args, pk, "timopel", "Timopel", TIMOPEL_SIZES, _timopel_config,
+                                   twins=(("medilix", _medilix_beside_timopel_config, "the Medilix design"),
+                                          ("logesun", _logesun_config, "the Logesun design")))
 
 
 def run_logesun(args, pk) -> dict:
@@ -836,8 +893,8 @@ def _fill_cache(storage) -> None:
 
 
 def run_design_beside_dense(args, pk, workload: str, design: str, sizes: dict, make_config,
-                            twin=("qwen3_dense", _dense_twin_config, "a Qwen3 dense model")) -> dict:
-    """Prefill and decode of a design beside another model of equal size: ``twin`` = (its label in the results,
+                            twins=(("qwen3_dense", _dense_twin_config, "a Qwen3 dense model"),)) -> dict:
+    """Prefill and decode of a design beside other models of equal size: each of ``twins`` = (its label in the results,
     its configuration for an entry of ``sizes``, its name in the metric's text)."""
     import torch
 
@@ -852,7 +909,7 @@ def run_design_beside_dense(args, pk, workload: str, design: str, sizes: dict, m
     clocks = ClockSampler().start()
     results = {}
     for size, z in sizes.items():
-        for arm, cfg in ((workload, make_config(z)), (twin[0], twin[1](z))):
+        for arm, cfg in ((workload, make_config(z)), *((label, config(z)) for label, config, _text in twins)):
             ops = CudaOps()
             model = build_model(cfg, RandomDeviceSource(expected_tensors_for(cfg), SEED, "cuda"), dtype="bfloat16",
                                 ops=ops)
@@ -873,7 +930,7 @@ def run_design_beside_dense(args, pk, workload: str, design: str, sizes: dict, m
             torch.cuda.empty_cache()
     first = results[f"w2048/{workload}"]
     return {
-        "metric": f"decode tok/s @ batch 8, ctx 1024 ({design} w2048 sizes, 4 layers, bf16); beside it {twin[2]} "
+        "metric": f"decode tok/s @ batch 8, ctx 1024 ({design} w2048 sizes, 4 layers, bf16); beside it {' and '.join(t[2] for t in twins)} "
                   "of equal size, and one 2048-token prefill of each",
         "value": first["decode_tok_s"], "unit": "tokens/s", "n_gpus": 1, "steps": K, "warmup": W,
         "ms_per_step": first["decode_ms_per_step"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
@@ -903,6 +960,8 @@ def run_workload_ours(args) -> dict:
         return run_tabisun(args, pk)
     if args.workload == "pevazen":
         return run_pevazen(args, pk)
+    if args.workload == "timopel":
+        return run_timopel(args, pk)
     cases = workload_prompts(args.workload, np)
     results, cfg, build_s, engine = {}, None, 0.0, None
     clocks = ClockSampler()
@@ -1160,7 +1219,7 @@ def main() -> int:
     args.warmup = max(3, args.warmup)
     if args.workload == "default":
         result = run_reference(args) if args.impl == "reference" else run_ours(args)
-    elif args.workload in ("logesun", "puladra", "medilix", "tabisun", "pevazen") and args.impl == "reference":
+    elif args.workload in ("logesun", "puladra", "medilix", "tabisun", "pevazen", "timopel") and args.impl == "reference":
         result = {"impl": "reference", "workload": args.workload,
                   "unavailable": "the reference has no model of this design (it serves Qwen3 dense only)"}
     else:

@@ -340,6 +340,99 @@ __global__ void qk_norm_store_kernel(T* __restrict__ proj, long row_stride, int 
   }
 }
 
+// The same without maps and rotation, with 16-byte accesses: sizes multiples of 8 up to 256, rows, columns and pages
+// 16-byte aligned.  1 << shift lanes per head, eight elements each; grid (tokens, blocks over one token's heads).
+template <typename T>
+__global__ void qk_norm_store_vec_kernel(T* __restrict__ proj, long row_stride, int nq, int nkv, int nv, int D, int Dv,
+                                         int k_start, int v_start, const float* __restrict__ q_w,
+                                         const float* __restrict__ k_w, float eps, const float* __restrict__ q_scale,
+                                         const T* __restrict__ v_first, long v_first_stride, float v_share,
+                                         const int* __restrict__ positions, const int* __restrict__ token_seq,
+                                         const int* __restrict__ block_table, int max_pages, T* __restrict__ kpages,
+                                         T* __restrict__ vpages, int ps, int shift, int write_kv) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int t = blockIdx.x;
+  const int u = blockIdx.y * blockDim.x + threadIdx.x;
+  const int lanes = 1 << shift;
+  const int hi = u >> shift, c = (u & (lanes - 1)) * 8;
+  const bool is_q = hi < nq, is_k = !is_q && hi < nq + nkv;
+  const bool live = hi < (write_kv ? nq + nkv + nv : nq);
+  T* row = proj + (long)t * row_stride;
+  long slot = -1;  // the token's row among all (page, head, place) rows
+  if (live && !is_q) {
+    const int p = positions[t];
+    if (p >= 0 && p / ps < max_pages) {
+      const int page = block_table[(long)token_seq[t] * max_pages + p / ps];
+      const int head = is_k ? hi - nq : hi - nq - nkv;
+      if (page >= 0) slot = ((long)page * (is_k ? nkv : nv) + head) * ps + (p % ps);
+    }
+  }
+  T* x = is_q ? row + (long)hi * D : row + k_start + (long)(hi - nq) * D;
+  const bool mine = live && (is_q || is_k) && c < D;
+  float a[8];
+#pragma unroll
+  for (int e = 0; e < 8; ++e) a[e] = 0.f;
+  if (mine) load8(x + c, a);
+  float ss = 0.f;
+#pragma unroll
+  for (int e = 0; e < 8; ++e) ss += a[e] * a[e];
+  for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if (mine) {
+    const float* w = is_q ? q_w : k_w;
+    if (w) {
+      const float rstd = rsqrtf(ss / (float)D + eps);
+      float wv[8];
+      load8(w + c, wv);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) a[e] = (a[e] * rstd) * wv[e];
+    }
+    if (is_q && q_scale) {
+      const float factor = q_scale[t];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) a[e] *= factor;
+    }
+    if (is_q)
+      store8(x + c, a);
+    else if (slot >= 0)
+      store8(kpages + slot * D + c, a);
+    return;
+  }
+  if (!live || is_q || is_k || slot < 0) return;
+  const int vh = hi - nq - nkv;
+  const T* v = row + v_start + (long)vh * Dv;
+  const T* f = v_first ? v_first + (long)t * v_first_stride + (long)vh * Dv : nullptr;
+  for (int d = c; d < Dv; d += lanes * 8) {
+    float b[8];
+    load8(v + d, b);
+    if (f) {
+      float fv[8];
+      load8(f + d, fv);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) b[e] = (1.f - v_share) * b[e] + v_share * fv[e];
+    }
+    store8(vpages + slot * Dv + d, b);
+  }
+}
+
+template <typename T>
+static int launch_qk_norm_store_vec(void* proj, long row_stride, int nq, int nkv, int nv, int D, int Dv, int k_start,
+                                    int v_start, const float* q_w, const float* k_w, float eps, const float* q_scale,
+                                    const void* v_first, long v_first_stride, float v_share, const int* positions,
+                                    const int* token_seq, const int* block_table, int max_pages, void* kpages,
+                                    void* vpages, int ps, int num_tokens, int write_kv, cudaStream_t stream) {
+  int shift = 0;
+  while ((8 << shift) < D) ++shift;
+  const long threads = (long)(write_kv ? nq + nkv + nv : nq) << shift;
+  const dim3 grid((unsigned)num_tokens, (unsigned)((threads + 127) / 128));
+  if (grid.y > 65535) return Q3_ERR_UNSUPPORTED;
+  return launch_pdl(qk_norm_store_vec_kernel<T>, grid, dim3(128), 0, stream, (T*)proj, row_stride, nq, nkv, nv, D, Dv,
+                    k_start, v_start, q_w, k_w, eps, q_scale, (const T*)v_first, v_first_stride, v_share, positions,
+                    token_seq, block_table, max_pages, (T*)kpages, (T*)vpages, ps, shift, write_kv) == cudaSuccess
+             ? Q3_OK
+             : Q3_ERR_LAUNCH;
+}
+
 Q3_EXPORT int q3_qk_norm_store(int dtype, void* proj, long row_stride, int nq, int nkv, int nv, int D, int Dv,
                                int k_start, int v_start, const float* q_w, const float* k_w, float eps, int maps,
                                const float* inv_freq, int rot_half, int pairing, float magnitude,
@@ -353,6 +446,19 @@ Q3_EXPORT int q3_qk_norm_store(int dtype, void* proj, long row_stride, int nq, i
   if (v_first && v_first_stride < (long)nv * Dv) return Q3_ERR_ARGUMENT;
   if (write_kv && (!token_seq || !block_table || !kpages || !vpages || max_pages < 1)) return Q3_ERR_ARGUMENT;
   if (num_tokens == 0) return Q3_OK;
+  if (maps == 1 && !inv_freq && D % 8 == 0 && Dv % 8 == 0 && D <= 256 && row_stride % 8 == 0 && k_start % 8 == 0 &&
+      v_start % 8 == 0 && v_first_stride % 8 == 0 && rk_aligned16(proj) && rk_aligned16(kpages) && rk_aligned16(vpages) &&
+      rk_aligned16(q_w) && rk_aligned16(k_w) && rk_aligned16(v_first)) {
+    if (dtype == Q3_DTYPE_F32)
+      return launch_qk_norm_store_vec<float>(proj, row_stride, nq, nkv, nv, D, Dv, k_start, v_start, q_w, k_w, eps, q_scale,
+                                             v_first, v_first_stride, v_share, positions, token_seq, block_table, max_pages,
+                                             kpages, vpages, ps, num_tokens, write_kv, stream);
+    if (dtype == Q3_DTYPE_BF16)
+      return launch_qk_norm_store_vec<bf16>(proj, row_stride, nq, nkv, nv, D, Dv, k_start, v_start, q_w, k_w, eps, q_scale,
+                                            v_first, v_first_stride, v_share, positions, token_seq, block_table, max_pages,
+                                            kpages, vpages, ps, num_tokens, write_kv, stream);
+    return Q3_ERR_ARGUMENT;
+  }
   constexpr int WARPS = 4;
   const size_t smem = (size_t)WARPS * D * sizeof(float);
   if (smem > 48 * 1024) return Q3_ERR_UNSUPPORTED;
