@@ -191,8 +191,12 @@ __device__ __forceinline__ int slices_of(const int* __restrict__ kv_lens, const 
 // operations, so both ways give the same bits).  Nothing the block reads before pdl_wait() is
 // written by a kernel of the same step, so the first key tiles are in flight while the
 // projection before this kernel is still finishing.
+// Blocks an SM has to hold (the cost model of the slice count assumes them): without the bound an option more in the
+// newest token's part can cost a block, and with it a sixth of a long step.
+template <int D> constexpr int resident_blocks() { return D == 64 ? 4 : D == 128 ? 3 : 1; }
+
 template <int D, bool FUSED>
-__global__ void __launch_bounds__(THREADS)
+__global__ void __launch_bounds__(THREADS, resident_blocks<D>())
 decode_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* kpages,
                         const bf16* vpages, const int* __restrict__ block_table, int max_pages,
                         const int* __restrict__ kv_lens, const int* __restrict__ cu_seqlens,
